@@ -6,7 +6,7 @@
 //   * the cache layout [page, 256, kv_heads, 128] makes the K (or V) rows of ALL kv heads of
 //     TILE consecutive tokens one contiguous TILE*kv_dim*2-byte span, so one CTA owns a token
 //     range of one sequence for every kv head and streams it with 1-D bulk async copies
-//     (cp.async.bulk -> SASS UBLKCP, the TMA unit) into an NSTAGE-deep shared-memory ring that
+//     (cp.async.bulk, the TMA unit) into an NSTAGE-deep shared-memory ring that
 //     completes on mbarriers; a dedicated producer warp issues, kv_heads consumer warps compute;
 //   * consumer warp w owns kv head w and both (GROUP) query heads that share it, so each K/V
 //     byte is read from HBM once and from shared memory once;

@@ -109,7 +109,7 @@ __device__ __forceinline__ void mbar_wait(uint64_t* bar, uint32_t parity) {
       "}"
       :: "r"(smem_u32(bar)), "r"(parity) : "memory");
 }
-// 1-D bulk copy global -> shared through the TMA unit (SASS: UBLKCP); completes on `bar`.
+// 1-D bulk copy global -> shared through the TMA unit; completes on `bar`.
 // dst/src 16-byte aligned, bytes a multiple of 16.
 __device__ __forceinline__ void bulk_g2s(void* smem_dst, const void* gsrc, uint32_t bytes, uint64_t* bar) {
   asm volatile(

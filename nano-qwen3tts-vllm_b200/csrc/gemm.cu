@@ -12,7 +12,7 @@
 //     "N" dimension (16..256), the accumulator D[128 features, Mpad] lives in TMEM;
 //   * W is re-packed ONCE at load time (b2tts_gemm_pack_weight) into the exact shared-memory
 //     image of a K-major SWIZZLE_128B operand tile, [n_tile][k_block] x 16 KiB, so one 1-D bulk
-//     async copy (cp.async.bulk -> UBLKCP, the TMA unit) per pipeline stage streams it, fully
+//     async copy (cp.async.bulk, the TMA unit) per pipeline stage streams it, fully
 //     contiguous in HBM, with no tensor map;
 //   * x (L2-resident, written by the previous kernel) is staged by 4 producer warps into the
 //     same swizzled layout (generic-proxy stores + fence.proxy.async);
