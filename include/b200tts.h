@@ -248,6 +248,8 @@ B2TTS_API int b2tts_frame_advance(const int64_t* code0, int eos_id, int32_t* act
  *                                              `rounding` as b2tts_silu_and_mul)
  *           B2TTS_GEMM_RELU_SQ   out[m, n]   = bf16(max(bf16(acc), 0)^2)      (squared-ReLU feed-forwards; single-GEMM
  *                                              entry points only)
+ *           B2TTS_GEMM_GELU_MUL  out[m, n/2] = bf16(gelu_tanh(gate) * up)     (B2TTS_PACK_GATE_UP weights; the float sums
+ *                                              feed the activation; single-GEMM entry points only)
  * splits: K-split = cluster size (1,2,4,8,16; 0 = choose so that tiles * splits fill the SMs); the
  * partial sums are exchanged through distributed shared memory and added in a fixed order.
  * splits = -2 / -4: the cluster splits the BATCH instead (m padded to 16 must be a multiple of 32 / 64, m <= 128):
@@ -261,6 +263,7 @@ B2TTS_API int b2tts_frame_advance(const int64_t* code0, int eos_id, int32_t* act
 #define B2TTS_GEMM_RESIDUAL 1
 #define B2TTS_GEMM_SILU_MUL 2
 #define B2TTS_GEMM_RELU_SQ  3
+#define B2TTS_GEMM_GELU_MUL 4
 #define B2TTS_PACK_PLAIN    0
 #define B2TTS_PACK_GATE_UP  1
 B2TTS_API int    b2tts_gemm_bf16_supported(int m, int n, int k);
@@ -432,19 +435,26 @@ B2TTS_API int b2tts_gather_gain_norm(const float* x, const int32_t* rows_idx, vo
                                      float eps, int dtype, void* stream);
 /* y <- max(y, 0)^2 in place. */
 B2TTS_API int b2tts_relu_sq(void* y, int64_t n, int dtype, void* stream);
+/* table[n, :] = [cos(positions[n] * freq[i]) for i < half | sin(.)], angles in float. */
+B2TTS_API int b2tts_rotary_table(const int32_t* positions, const float* freq, float* table, int n, int half, void* stream);
 /* Short causal convolution over time on every channel of the merged projection u [n, C] = [q | k | v]
  * (C = heads*dim + kv_heads*dim + kv_heads*vdim; conv_w [C, taps] float, tap taps-1 is the token itself), then RMS norm
  * per head over dim with q_norm_w / k_norm_w [dim] for q and k; q goes to q_out [n, heads*dim], k and v to their cache
  * slot (slot_mapping[n]).  Token n belongs to batch row tok_seq[n] at position positions[n]; row b brings seq_len[b]
  * tokens starting at batch index seq_start[b] and position seq_pos0[b], and owns state slot seq_slot[b]:
  * state [slots, taps-1, C] holds the last taps-1 projections of the sequence (oldest first) and is advanced by this
- * call.  Positions before 0 read as zero whatever the slot holds, so a slot needs no clearing between owners. */
+ * call.  Positions before 0 read as zero whatever the slot holds, so a slot needs no clearing between owners.
+ * rot_dims > 0: between convolution and norm, coordinate i < rot_dims/2 of every q and k head is paired with i + rot_dims/2 and
+ * turned by the angles of rot [n, rot_dims] (cosines, then sines: b2tts_rotary_table).  Norm weights may be null (none).
+ * flags: 1 = round the convolution's q and k to the activation type before the norm; 2 = v is divided by its head's root
+ * mean square too (no weight). */
 B2TTS_API int b2tts_conv_headnorm_kvwrite(const void* u, int64_t u_stride, const float* conv_w, void* state,
                                           const int32_t* tok_seq, const int32_t* positions, const int32_t* seq_start,
                                           const int32_t* seq_pos0, const int32_t* seq_len, const int32_t* seq_slot,
                                           const int32_t* slot_mapping, const float* q_norm_w, const float* k_norm_w,
                                           void* q_out, void* k_cache, void* v_cache, int n_tokens, int n_seqs, int heads,
-                                          int kv_heads, int dim, int vdim, int taps, float eps, int dtype, void* stream);
+                                          int kv_heads, int dim, int vdim, int taps, float eps,
+                                          const float* rot, int rot_dims, int flags, int dtype, void* stream);
 /* Sliding-window attention with un-normalised sigmoid weights and a logarithmic distance bias over the paged cache:
  * out[i, h] = sum_{0 <= i-j < window} sigmoid(q_ih . k_jg * scale - r1[h] * ln(1 + r2[h] * (i-j)) + pb[h]) * v_jg.
  * q [n, heads*dim], caches [slots, kv_heads*dim] / [slots, kv_heads*vdim], out [n, heads*vdim]; key j of batch row b lives
@@ -627,6 +637,33 @@ B2TTS_API int b2tts_diff_combine(const void* maps, void* out, float lambda, floa
                                  int maps_f32, int dtype, void* stream);
 /* In place: y <- cap * tanh(y / cap). */
 B2TTS_API int b2tts_tanh_cap(float* y, int64_t n, float cap, void* stream);
+
+/* ---- decoders with gated residuals and fixed-decay retention (csrc/gated_ops.cu, csrc/retention.cu) ----
+ * x[r] (init != 0: starting from zero) += sigmoid(z[r * ldz + c] + zb[c]) * y[r] (z null: y as it is; y null: nothing), then += row
+ * index[r] of `table` (null: nothing), then += add[c] (null: nothing); h[r] = x[r] / sqrt(mean(x[r]^2) + eps) * w when h != null. */
+B2TTS_API int b2tts_gated_residual(float* x, const void* y, const void* z, int64_t ldz, const float* zb, const void* table,
+                                   const int32_t* index, int table_rows, const float* add, const float* w, void* h, int rows,
+                                   int cols, int init, float eps, int dtype, void* stream);
+/* y[r, c] = gelu_tanh(gu[r, c]) * gu[r, ff + c], gu [rows, 2 ff]; gelu_tanh(z) = z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))). */
+B2TTS_API int b2tts_gelu_mul(const void* gu, void* y, int64_t rows, int ff, int dtype, void* stream);
+/* Recurrence with a fixed decay per head on float inputs, state [slots, heads, dim, vdim] float: S <- head_decay[h] S + k v^T;
+ * out[t, h] = S^T q.  rows: 0 every sequence, 1 only those with more than one new token, 2 only one-token ones. */
+B2TTS_API int b2tts_fixed_decay_scan(const float* q, int64_t ldq, const float* k, int64_t ldk, const float* v, int64_t ldv,
+                                     const float* head_decay, float* state, float* out, const int32_t* seq_start,
+                                     const int32_t* seq_pos0, const int32_t* seq_len, const int32_t* seq_slot, int n_tokens,
+                                     int n_seqs, int heads, int dim, int vdim, int rows, void* stream);
+/* Retention: q and k [rows, heads*dim] rotated (coordinate i with i + rot_dims/2) by rot [rows, rot_dims] (b2tts_rotary_table;
+ * rot_dims 0: not rotated), k also times k_scale; S <- decay[h] S + k v^T, o = S^T q (state as above); then out[t, h] = o /
+ * sqrt(mean over vdim of o^2 + eps) * silu(gate[t * ldg + h * vdim + c]).  q, k, v, gate and out have the activation type.  Scratch, as
+ * b2tts_retention_scratch says: 0 none, 1 `o` [rows, heads*vdim] float, 2 also `qkv` [rows, 2*heads*dim + heads*vdim] float
+ * (aligned: q, k, v on 16-byte boundaries with row strides of whole 8 elements).  path: 0 chosen by shape, 1 the
+ * token-by-token scan for everything, 2 insist on the tensor-core kernel for prompt portions. */
+B2TTS_API int b2tts_retention(const void* q, int64_t ldq, const void* k, int64_t ldk, const void* v, int64_t ldv, const float* rot,
+                              int rot_dims, const float* decay, float k_scale, float* state, const void* gate, int64_t ldg, float* o,
+                              float* qkv, void* out, const int32_t* seq_start, const int32_t* seq_pos0, const int32_t* seq_len,
+                              const int32_t* seq_slot, int n_tokens, int n_seqs, int max_new, int heads, int dim, int vdim, float eps,
+                              int dtype, int path, void* stream);
+B2TTS_API int b2tts_retention_scratch(int dim, int vdim, int max_new, int rot_dims, int aligned, int dtype, int path);
 
 #ifdef __cplusplus
 }

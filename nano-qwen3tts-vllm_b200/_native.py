@@ -83,7 +83,13 @@ def _load():
         "b2tts_residual_norm": (I, [P, P, P, P, P, I, F, P, P, I, I, F, I, P]),
         "b2tts_gather_gain_norm": (I, [P, P, P, P, I, I, F, I, P]),
         "b2tts_relu_sq": (I, [P, L, I, P]),
-        "b2tts_conv_headnorm_kvwrite": (I, [P, L, P, P, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, I, P]),
+        "b2tts_conv_headnorm_kvwrite": (I, [P, L, P, P, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, P, I, I, I, P]),
+        "b2tts_rotary_table": (I, [P, P, P, I, I, P]),
+        "b2tts_gated_residual": (I, [P, P, P, L, P, P, P, I, P, P, P, I, I, I, F, I, P]),
+        "b2tts_gelu_mul": (I, [P, P, L, I, I, P]),
+        "b2tts_fixed_decay_scan": (I, [P, L, P, L, P, L, P, P, P, P, P, P, P, I, I, I, I, I, I, P]),
+        "b2tts_retention": (I, [P, L, P, L, P, L, P, I, P, F, P, P, L, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, P]),
+        "b2tts_retention_scratch": (I, [I, I, I, I, I, I, I]),
         "b2tts_window_sigmoid_attn": (I, [P, P, P, P, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, I, P]),
         "b2tts_moe_route": (I, [P, P, P, P, P, P, I, I, I, I, F, P, I, I, P]),
         "b2tts_embed_scale": (I, [P, P, P, I, I, I, F, I, P]),
@@ -449,7 +455,7 @@ def frame_advance(code0, eos_id, active, seq_lens, gen_step, frames_done, extra_
 
 
 # ------------------------------------------------------------------------------------------ a7
-GEMM_BIAS, GEMM_RESIDUAL, GEMM_SILU_MUL, GEMM_RELU_SQ = 0, 1, 2, 3
+GEMM_BIAS, GEMM_RESIDUAL, GEMM_SILU_MUL, GEMM_RELU_SQ, GEMM_GELU_MUL = 0, 1, 2, 3, 4
 PACK_PLAIN, PACK_GATE_UP = 0, 1
 GEMM_MAX_M = 1 << 16        # any batch: rows beyond 128 run as 128-row chunks of the same kernel (gemm.cu)
 GEMM_CHAIN_MAX_M = 128
@@ -494,7 +500,7 @@ def gemm_ssq_slots(m: int, n: int, k: int, splits: int = 0) -> int:
 def gemm_bf16(x, packed, n, bias=None, residual=None, epilogue=GEMM_BIAS, rounding=ROUND_EAGER, out=None,
               splits=0, pdl=False, norm_weight=None, ssq_in=None, eps=1e-6, ssq_out=None, prefetch=None):
     """y = epilogue(x[M,K] @ W[N,K]^T) with W pre-packed by ``gemm_pack_weight``; bf16 in/out, fp32
-    accumulation in TMEM.  GEMM_SILU_MUL returns [M, N/2]; GEMM_RESIDUAL may write in place (out=residual).
+    accumulation in TMEM.  GEMM_SILU_MUL and GEMM_GELU_MUL return [M, N/2]; GEMM_RESIDUAL may write in place (out=residual).
     ``norm_weight`` + ``ssq_in`` [M, slots] fp32: x is normalised (RMSNorm) while it is staged.
     ``ssq_out`` [M, gemm_ssq_slots(n, k, splits)] fp32 receives the row sums of squares of the output.
     ``prefetch``: the packed image of the NEXT projection's weight - pulled into L2 while this GEMM runs."""
@@ -502,7 +508,7 @@ def gemm_bf16(x, packed, n, bias=None, residual=None, epilogue=GEMM_BIAS, roundi
     m, k = x.shape
     if x.stride(1) != 1:
         x = x.contiguous()
-    cols = n // 2 if epilogue == GEMM_SILU_MUL else n
+    cols = n // 2 if epilogue in (GEMM_SILU_MUL, GEMM_GELU_MUL) else n
     if out is None:
         out = torch.empty(m, cols, dtype=BF16, device=x.device)
     if residual is not None:
@@ -757,17 +763,33 @@ def relu_sq_(y):
     return y
 
 
+CONV_ROUND, CONV_UNIT_V = 1, 2
+
+
+def rotary_table(positions, freq):
+    """[n, 2 * len(freq)] float: cosines, then sines, of positions[n] * freq[i]."""
+    _cuda(positions, I32, "positions"); _cuda(freq, F32, "freq")
+    out = torch.empty(positions.shape[0], 2 * freq.shape[0], dtype=F32, device=positions.device)
+    _check(_load().b2tts_rotary_table(positions.data_ptr(), freq.data_ptr(), out.data_ptr(), positions.shape[0], freq.shape[0], _stream()),
+           "rotary_table")
+    return out
+
+
 def conv_headnorm_kvwrite(u, conv_w, state, lay, q_norm_w, k_norm_w, q_out, k_cache, v_cache, heads, kv_heads, dim, vdim,
-                          taps, eps):
+                          taps, eps, rot=None, flags=CONV_ROUND):
     """``lay``: the step's device layout (tok_seq, positions, seq_start, seq_pos0, seq_len, seq_slot, slot_mapping as
-    int32 tensors, n_tokens, n_seqs)."""
+    int32 tensors, n_tokens, n_seqs).  ``rot``: the step's ``rotary_table`` - q and k heads are rotated between convolution
+    and norm; norm weights None: none; ``flags``: CONV_ROUND rounds the convolved q and k to the activation type before the
+    norm, CONV_UNIT_V divides v by its head's root mean square."""
     dt = _act(u, "u")
-    assert k_cache.dtype == u.dtype and v_cache.dtype == u.dtype and q_out.dtype == u.dtype
+    assert k_cache.dtype == u.dtype and v_cache.dtype == u.dtype and q_out.dtype == u.dtype and u.stride(1) == 1
+    assert rot is None or (rot.dtype == F32 and rot.is_contiguous() and rot.shape[0] >= lay.n_tokens)
     _check(_load().b2tts_conv_headnorm_kvwrite(
         u.data_ptr(), u.stride(0), conv_w.data_ptr(), _ptr(state), lay.tok_seq.data_ptr(), lay.positions.data_ptr(),
         lay.seq_start.data_ptr(), lay.seq_pos0.data_ptr(), lay.seq_len.data_ptr(), lay.seq_slot.data_ptr(),
-        lay.slot_mapping.data_ptr(), q_norm_w.data_ptr(), k_norm_w.data_ptr(), q_out.data_ptr(), k_cache.data_ptr(),
-        v_cache.data_ptr(), lay.n_tokens, lay.n_seqs, heads, kv_heads, dim, vdim, taps, eps, dt, _stream()),
+        lay.slot_mapping.data_ptr(), _ptr(q_norm_w), _ptr(k_norm_w), q_out.data_ptr(), k_cache.data_ptr(),
+        v_cache.data_ptr(), lay.n_tokens, lay.n_seqs, heads, kv_heads, dim, vdim, taps, eps, _ptr(rot),
+        0 if rot is None else rot.shape[1], flags, dt, _stream()),
         "conv_headnorm_kvwrite")
 
 
@@ -1005,10 +1027,12 @@ GATE_SIGMOID, GATE_SILU = 0, 1
 
 def gated_group_norm(y, gate, w, groups, gate_act, gate_first, eps, out):
     """y [n, C] float -> out [n, C]: gate and RMS norm in ``groups`` parts, weight w[c mod len(w)]."""
-    _cuda(y, F32, "y"); _cuda(w, F32, "w")
+    _cuda(y, F32, "y")
+    assert w is None or w.dtype == F32
     dt = _act(out, "out")
     assert y.is_contiguous() and (gate is None or (gate.dtype == out.dtype and gate.stride(1) == 1))
-    _check(_load().b2tts_gated_group_norm(y.data_ptr(), _ptr(gate), 0 if gate is None else gate.stride(0), w.data_ptr(), w.numel(),
+    _check(_load().b2tts_gated_group_norm(y.data_ptr(), _ptr(gate), 0 if gate is None else gate.stride(0), _ptr(w),
+                                          0 if w is None else w.numel(),
                                           groups, gate_act, int(gate_first), eps, out.data_ptr(), y.shape[0], y.shape[1], dt, _stream()),
            "gated_group_norm")
 
@@ -1123,3 +1147,57 @@ def matrix_memory_scan(q, k, v, ig, fg, i_bias, f_bias, cap, state, state_nm, ga
                                             i_bias.data_ptr(), f_bias.data_ptr(), cap, state.data_ptr(), state_nm.data_ptr(),
                                             gates.data_ptr(), out.data_ptr(), *_seq_args(lay, True), heads, dim, vdim, dt, _stream()),
            "matrix_memory_scan")
+
+
+# ------------------------------------------------------------------------------------------ gated residuals, retention
+def gated_residual(x, *, y=None, z=None, zb=None, table=None, index=None, add=None, w=None, init=False, eps=1e-6, dtype=None):
+    """x (float [n, cols], in place; ``init``: starts from zero) += sigmoid(z + zb) * y, += table[index], += add; returns
+    x / sqrt(mean(x^2) + eps) * w in the activation type when ``w`` is given.  ``z``: a column slice [n, cols]."""
+    _cuda(x, F32, "x")
+    n, cols = x.shape
+    dtype = dtype or next(t.dtype for t in (y, table) if t is not None)
+    assert x.is_contiguous()
+    for t in (y, table):
+        assert t is None or (t.dtype == dtype and t.is_contiguous() and t.shape[1] == cols)
+    assert z is None or (z.dtype == dtype and z.stride(1) == 1 and z.shape == x.shape)
+    for t in (zb, add, w):
+        assert t is None or (t.dtype == F32 and t.is_contiguous() and t.numel() == cols)
+    h = torch.empty(n, cols, dtype=dtype, device=x.device) if w is not None else None
+    _check(_load().b2tts_gated_residual(x.data_ptr(), _ptr(y), _ptr(z), 0 if z is None else z.stride(0), _ptr(zb), _ptr(table), _ptr(index),
+                                        0 if table is None else table.shape[0], _ptr(add), _ptr(w), _ptr(h), n, cols, int(init), eps,
+                                        DTYPE_CODE[dtype], _stream()), "gated_residual")
+    return h
+
+
+def gelu_mul(gu, out=None):
+    """gu [rows, 2 ff] = [gate | up] -> gelu_tanh(gate) * up."""
+    dt = _act(gu, "gu")
+    ff = gu.shape[1] // 2
+    if out is None:
+        out = torch.empty(gu.shape[0], ff, dtype=gu.dtype, device=gu.device)
+    _check(_load().b2tts_gelu_mul(gu.data_ptr(), out.data_ptr(), gu.shape[0], ff, dt, _stream()), "gelu_mul")
+    return out
+
+
+RETENTION_AUTO, RETENTION_SCAN, RETENTION_TENSOR = 0, 1, 2
+
+
+def retention(q, k, v, rot, decay, k_scale, state, gate, out, lay, heads, dim, vdim, eps, path=RETENTION_AUTO):
+    """q, k [n, heads*dim], v, gate [n, heads*vdim]: column slices with unit column stride; ``rot``: the step's
+    ``rotary_table`` (None: no rotation); decay float [heads]; state float [slots, heads, dim, vdim] advances; out [n, heads*vdim] =
+    head_rms_norm(S^T q) * silu(gate)."""
+    dt = _act(out, "out")
+    _cuda(state, F32, "state"); _cuda(decay, F32, "decay")
+    for t in (q, k, v, gate):
+        assert t.dtype == out.dtype and t.stride(1) == 1
+    assert state.is_contiguous() and (rot is None or (rot.dtype == F32 and rot.is_contiguous()))
+    rd = 0 if rot is None else rot.shape[1]
+    aligned = all(t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0 for t in (q, k, v))
+    need = _load().b2tts_retention_scratch(dim, vdim, lay.max_new, rd, int(aligned), dt, path)
+    n = out.shape[0]
+    o = torch.empty(n, heads * vdim, dtype=F32, device=out.device) if need else None
+    qkv = torch.empty(n, heads * (2 * dim + vdim), dtype=F32, device=out.device) if need > 1 else None
+    _check(_load().b2tts_retention(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), _ptr(rot), rd,
+                                   decay.data_ptr(), k_scale, state.data_ptr(), gate.data_ptr(), gate.stride(0), _ptr(o), _ptr(qkv),
+                                   out.data_ptr(), *_seq_args(lay, True), lay.max_new, heads, dim, vdim, eps, dt, path, _stream()),
+           "retention")

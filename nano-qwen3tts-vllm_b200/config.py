@@ -357,6 +357,9 @@ class SinkAttentionSpec:
     softcap: float = 0.0           # c > 0: scaled scores become c tanh(s / c)
     keep_first: int = 0            # keys below this position stay visible behind the mask
     sink: str = "learned"          # "learned": exp(sink_h) in the denominator;  "zero": exp(0);  "none": an ordinary softmax
+    conv: int = 0                  # taps of a short causal convolution on every channel of q, k and v (0: none)
+    unit_qk: bool = False          # after rotation every q and k head is divided by its root mean square (no weight)
+    unit_v: bool = False           # so is every value head
 
 
 @dataclass
@@ -672,6 +675,107 @@ class TeberaxConfig:
                "layers": layers}
         if self.logit_softcap:
             out["logit_softcap"] = self.logit_softcap
+        return out
+
+
+@dataclass
+class RetentionSpec:
+    """Linear attention with a fixed decay per head (no softmax, no denominator): rotated q and k, a matrix state per head,
+    read-outs divided by their root mean square, a SiLU gate."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: list
+    rot: HalfRotarySpec | None = None
+
+
+@dataclass
+class ZekivikLayerSpec:
+    type: str                      # "attention" | "retention"
+    mixer: object                  # SinkAttentionSpec | RetentionSpec
+    mlp: FeedForwardSpec | None
+    raw: dict = field(default_factory=dict, repr=False)      # the layer's entry as read (kept for to_dict)
+
+
+@dataclass
+class ZekivikConfig:
+    """``config.json`` of a Zekivik checkpoint: a decoder-only token model over one 32-bit residual stream whose sublayers
+    pass an element-wise gate before they join it.  Layers are listed one by one with their own sizes: causal softmax
+    attention over convolved, rotated and unit-normed heads, or retention with a fixed decay per head; feed-forwards are
+    GELU-gated or absent.  ``loop`` repeats a range of layers with the same weights, each pass over a cache and state of
+    its own; a pass starts with a vector of its own, a later one also with the token's embedding again."""
+    architecture: str
+    vocab: int
+    width: int
+    norm_eps: float
+    layers: list
+    loop: dict | None              # {"start", "stop", "times"}
+    max_positions = None           # positions enter through rotations only: no table bounds them
+
+    page_multiple = 16
+
+    @staticmethod
+    def _rot(r: dict | None, dim: int, i: int) -> HalfRotarySpec | None:
+        if not r or not int(r["dims"]):
+            return None
+        rot = HalfRotarySpec(int(r["dims"]), float(r["base"]))
+        if rot.dims % 2 or not 0 < rot.dims <= dim:
+            raise ValueError(f"layer {i}: {rot.dims} rotated coordinates in a head of {dim}")
+        return rot
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "ZekivikConfig":
+        layers = []
+        for i, ld in enumerate(d["layers"]):
+            kind, m = ld["type"], ld["mixer"]
+            if kind == "attention":
+                mixer = SinkAttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                                          mask_kind="window", mask_size=0, scale=float(m["scale"]), rot=cls._rot(m.get("rot"), int(m["dim"]), i),
+                                          gate=True, sink="none", conv=int(m["conv"]), unit_qk=True, unit_v=True)
+                if mixer.heads % mixer.kv_heads:
+                    raise ValueError(f"layer {i}: {mixer.heads} heads over {mixer.kv_heads} key/value heads")
+                if mixer.conv < 1:
+                    raise ValueError(f"layer {i}: a convolution of {mixer.conv} taps")
+            elif kind == "retention":
+                mixer = RetentionSpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), decay=[float(x) for x in m["decay"]],
+                                      rot=cls._rot(m.get("rot"), int(m["dim"]), i))
+                if len(mixer.decay) != mixer.heads:
+                    raise ValueError(f"layer {i}: {len(mixer.decay)} decays for {mixer.heads} heads")
+            else:
+                raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+            f = ld.get("mlp")
+            mlp = None
+            if f is not None:
+                if f["kind"] != "dense":
+                    raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
+                mlp = FeedForwardSpec("dense", int(f["ff"]), act="gelu_gate")
+            layers.append(ZekivikLayerSpec(kind, mixer, mlp, raw=ld))
+        lp = d.get("loop")
+        loop = {k: int(lp[k]) for k in ("start", "stop", "times")} if lp else None
+        if loop is not None and not (0 <= loop["start"] < loop["stop"] <= len(layers) and loop["times"] >= 1):
+            raise ValueError(f"loop {loop} does not fit {len(layers)} layers")
+        return cls(architecture=d["architecture"], vocab=int(d["vocab"]), width=int(d["width"]), norm_eps=float(d["norm"]["eps"]),
+                   layers=layers, loop=loop)
+
+    @classmethod
+    def from_pretrained(cls, model_dir: str) -> "ZekivikConfig":
+        with open(os.path.join(model_dir, "config.json")) as f:
+            return cls.from_dict(json.load(f))
+
+    def runs(self) -> list[tuple[int, int | None]]:
+        """(layer index, number of the pass that starts right before it or None) of every layer run, in order."""
+        n = len(self.layers)
+        if not self.loop:
+            return [(i, None) for i in range(n)]
+        a, b, times = self.loop["start"], self.loop["stop"], self.loop["times"]
+        looped = [(i, t if i == a else None) for t in range(times) for i in range(a, b)]
+        return [(i, None) for i in range(a)] + looped + [(i, None) for i in range(b, n)]
+
+    def to_dict(self) -> dict:
+        out = {"architecture": self.architecture, "vocab": self.vocab, "width": self.width, "norm": {"eps": self.norm_eps},
+               "layers": [dict(l.raw) for l in self.layers]}
+        if self.loop:
+            out["loop"] = dict(self.loop)
         return out
 
 

@@ -424,6 +424,15 @@ gemm_stream_kernel(const GemmParams p, const __grid_constant__ CUtensorMap tmap_
         stg_v2(p.out + (int64_t)(row0 + m) * p.out_stride + (n >> 1), w);
         return 0.f;
       }
+      if (p.epilogue == B2TTS_GEMM_GELU_MUL) {                      // same packing; the float sums feed the activation
+        float o[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) o[j] = gelu_tanh_f(acc[j]) * acc[4 + j];
+        uint2 w;
+        w.x = pack_bf16(o[0], o[1]); w.y = pack_bf16(o[2], o[3]);
+        stg_v2(p.out + (int64_t)(row0 + m) * p.out_stride + (n >> 1), w);
+        return 0.f;
+      }
       if (p.epilogue == B2TTS_GEMM_BIAS && p.bias) {
         const uint4 bw = have_pre ? pre : ldg_v4(p.bias + n);
         acc[0] += bf16lo(bw.x); acc[1] += bf16hi(bw.x); acc[2] += bf16lo(bw.y); acc[3] += bf16hi(bw.y);
@@ -693,15 +702,16 @@ static int gemm_impl(const char* what, const void* x, int64_t x_row_stride, cons
              "%s: m=%d (1..%d), n=%d (multiple of %d), k=%d (multiple of %d)", what, m, G_MAX_ROWS, n, G_BN, k, G_BK);
   B2_REQUIRE(x && w_packed && out, B2TTS_EINVAL, "%s: null pointer", what);
   B2_REQUIRE(epilogue == B2TTS_GEMM_BIAS || epilogue == B2TTS_GEMM_RESIDUAL || epilogue == B2TTS_GEMM_SILU_MUL ||
-                 epilogue == B2TTS_GEMM_RELU_SQ, B2TTS_EINVAL, "%s: epilogue %d", what, epilogue);
+                 epilogue == B2TTS_GEMM_RELU_SQ || epilogue == B2TTS_GEMM_GELU_MUL, B2TTS_EINVAL, "%s: epilogue %d", what, epilogue);
   B2_REQUIRE(epilogue != B2TTS_GEMM_RESIDUAL || residual, B2TTS_EINVAL, "%s: residual epilogue without residual", what);
   B2_REQUIRE(aligned16(x) && aligned16(w_packed) && aligned16(out) && x_row_stride % 8 == 0 && out_row_stride % 4 == 0 &&
-                 (epilogue == B2TTS_GEMM_SILU_MUL || out_row_stride % 8 == 0) &&
+                 (epilogue == B2TTS_GEMM_SILU_MUL || epilogue == B2TTS_GEMM_GELU_MUL || out_row_stride % 8 == 0) &&
                  (!bias || aligned16(bias)) && (!residual || (aligned16(residual) && residual_row_stride % 8 == 0)),
              B2TTS_EALIGN, "%s: pointers / strides must be 16-byte aligned", what);
   B2_REQUIRE(!norm_weight || (ssq_in && ssq_in_slots > 0 && aligned16(norm_weight) && aligned16(ssq_in)), B2TTS_EINVAL,
              "%s: fused norm needs ssq_in with >= 1 slot per row (16-byte aligned)", what);
-  B2_REQUIRE(!ssq_out || epilogue != B2TTS_GEMM_SILU_MUL, B2TTS_EINVAL, "%s: ssq_out with the SiLU*mul epilogue", what);
+  B2_REQUIRE(!ssq_out || (epilogue != B2TTS_GEMM_SILU_MUL && epilogue != B2TTS_GEMM_GELU_MUL), B2TTS_EINVAL,
+             "%s: ssq_out with a gated epilogue", what);
   GemmParams p{};
   p.x = static_cast<const __nv_bfloat16*>(x);
   p.x_stride = x_row_stride;

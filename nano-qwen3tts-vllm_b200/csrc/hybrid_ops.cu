@@ -427,7 +427,7 @@ __global__ void conv_state_advance_kernel(const T* __restrict__ u, int64_t ldu, 
 
 // ------------------------------------------------------------------ gate + grouped RMS norm on a branch output
 // One block per (row, group): the row y [cols] (float) is cut into `groups` equal consecutive parts; each part is divided
-// by its own root mean square and multiplied by w[c mod w_len]; the gate act(gate[r, c]) multiplies y before the norm
+// by its own root mean square and multiplied by w[c mod w_len] (w null: by one); the gate act(gate[r, c]) multiplies y before the norm
 // (gate_first) or the normed result.  act 0: sigmoid, 1: SiLU.
 template <typename T>
 __global__ void __launch_bounds__(ROW_THREADS)
@@ -456,8 +456,9 @@ gated_group_norm_kernel(const float* __restrict__ y, const T* __restrict__ gate,
       g = to_f(gr[c]);
       g = act == 0 ? sigmoid_f(g) : silu_f(g);
     }
-    if (gate_first) v = v * g * inv * w[(c0 + c) % w_len];
-    else v = v * inv * w[(c0 + c) % w_len] * g;
+    const float ww = w != nullptr ? w[(c0 + c) % w_len] : 1.f;
+    if (gate_first) v = v * g * inv * ww;
+    else v = v * inv * ww * g;
     o[c] = from_f<T>(v);
   }
 }
@@ -509,7 +510,7 @@ gated_group_norm_vec4_kernel(const float* __restrict__ y, const T* __restrict__ 
   T* o = out + r * cols + c0;
   auto emit = [&](int c, const float4& v, const float4& g) {
     const int wc = (c0 + c) % w_len;                       // w_len is a multiple of four here
-    const float4 ww = *reinterpret_cast<const float4*>(w + wc);
+    const float4 ww = w != nullptr ? *reinterpret_cast<const float4*>(w + wc) : make_float4(1.f, 1.f, 1.f, 1.f);
     float4 res = make_float4(v.x * inv * ww.x, v.y * inv * ww.y, v.z * inv * ww.z, v.w * inv * ww.w);
     if (!gate_first) { res.x *= g.x; res.y *= g.y; res.z *= g.z; res.w *= g.w; }
     store4<T>(o + c, res);
@@ -566,7 +567,7 @@ gated_group_norm_warp_kernel(const float* __restrict__ y, const T* __restrict__ 
     for (int it = 0; it < GNW_KEEP; ++it) {
       const int c = (lane + it * 32) * 4;
       if (c < gs) {
-        const float4 ww = *reinterpret_cast<const float4*>(w + (c0 + c) % w_len);
+        const float4 ww = w != nullptr ? *reinterpret_cast<const float4*>(w + (c0 + c) % w_len) : make_float4(1.f, 1.f, 1.f, 1.f);
         float4 res = make_float4(kv[it].x * inv * ww.x, kv[it].y * inv * ww.y, kv[it].z * inv * ww.z, kv[it].w * inv * ww.w);
         if (!gate_first) { res.x *= kg[it].x; res.y *= kg[it].y; res.z *= kg[it].z; res.w *= kg[it].w; }
         store4<T>(o + c, res);
@@ -726,16 +727,17 @@ extern "C" int b2tts_short_conv_act(const void* u, int64_t ldu, int c_off, const
 extern "C" int b2tts_gated_group_norm(const float* y, const void* gate, int64_t ldg, const float* w, int w_len, int groups,
                                       int gate_act, int gate_first, float eps, void* out, int rows, int cols, int dtype,
                                       void* stream) {
-  B2_REQUIRE(rows >= 0 && cols > 0 && groups > 0 && cols % groups == 0 && w_len > 0, B2TTS_EINVAL,
+  B2_REQUIRE(rows >= 0 && cols > 0 && groups > 0 && cols % groups == 0 && (!w || w_len > 0), B2TTS_EINVAL,
              "gated_group_norm: rows=%d cols=%d groups=%d", rows, cols, groups);
   B2_REQUIRE(gate_act == 0 || gate_act == 1, B2TTS_EINVAL, "gated_group_norm: gate_act %d", gate_act);
   B2_REQUIRE(B2_ROW_DTYPE_OK(dtype), B2TTS_EINVAL, "gated_group_norm: dtype %d", dtype);
   if (rows == 0) return B2TTS_OK;
-  B2_REQUIRE(y && w && out, B2TTS_EINVAL, "gated_group_norm: null pointer");
+  B2_REQUIRE(y && out, B2TTS_EINVAL, "gated_group_norm: null pointer");
+  if (w == nullptr) w_len = 4;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int gs = cols / groups;
   const dim3 grid(rows, groups);
-  const bool vec4 = gs % 4 == 0 && w_len % 4 == 0 && ldg % 4 == 0 && aligned16(y) && aligned16(w) && aligned16(out) &&
+  const bool vec4 = gs % 4 == 0 && w_len % 4 == 0 && ldg % 4 == 0 && aligned16(y) && (!w || aligned16(w)) && aligned16(out) &&
                     (!gate || aligned16(gate));
   if (vec4 && groups > 1 && gs <= 4 * GNW_KEEP * 32) {
     const int threads = 32 * std::min(groups, ROW_THREADS / 32);

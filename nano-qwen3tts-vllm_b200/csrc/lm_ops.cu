@@ -119,6 +119,21 @@ __global__ void relu_sq_kernel(T* __restrict__ y, size_t n) {
   }
 }
 
+// ------------------------------------------------------------------ cosines and sines of a step's positions
+// table[n, i] = cos(position[n] * freq[i]), table[n, half + i] = sin(.), i < half; the angle is formed in float.  One table
+// per step serves every layer with the same frequencies.
+__global__ void rotary_table_kernel(const int32_t* __restrict__ positions, const float* __restrict__ freq, float* __restrict__ table,
+                                    int n, int half) {
+  const size_t idx = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (idx >= static_cast<size_t>(n) * half) return;
+  const size_t t = idx / half;
+  const int i = static_cast<int>(idx % half);
+  float sn, cs;
+  sincosf(static_cast<float>(positions[t]) * freq[i], &sn, &cs);
+  table[t * 2 * half + i] = cs;
+  table[t * 2 * half + half + i] = sn;
+}
+
 // ------------------------------------------------------------------ short convolution + head norm + paged K/V write
 // One warp per (token, head slot); head slots are the H query heads, then the G key heads, then the G value heads of the
 // merged projection row u[n] = [q | k | v].  Tap j of the token at position p reads the projection of position
@@ -126,7 +141,20 @@ __global__ void relu_sq_kernel(T* __restrict__ y, size_t n) {
 // state (its last taps - 1 projections, oldest first) when it came earlier, zero before the sequence's start.
 constexpr int CONV_WARPS = 8;
 constexpr int CONV_MAX_PER_LANE = 8;       // head sizes up to 256
-constexpr int CONV_MAX_TAPS = 8;
+constexpr int CONV_MAX_TAPS = 16;
+
+// What happens to a head between the convolution and the store.  Default (CONV_ROUND): q and k are rounded to T, divided
+// by the root mean square of the head and multiplied by their weight; v is stored as it is.
+//   rot, rot_dims   coordinate i < rot_dims / 2 of a q / k head is paired with i + rot_dims / 2 and the pair turned by the
+//                   token's angle, before the norm: rot [n, rot_dims] holds the cosines, then the sines (b2tts_rotary_table)
+//   CONV_UNIT_V     v is divided by the root mean square of its head too, without a weight
+//   without CONV_ROUND the convolution's float results feed rotation and norm unrounded
+struct ConvHeadOps {
+  const float* rot;
+  int rot_dims;
+  int flags;
+};
+constexpr int CONV_ROUND = 1, CONV_UNIT_V = 2;
 
 template <typename T>
 __global__ void __launch_bounds__(CONV_WARPS * 32)
@@ -137,7 +165,8 @@ conv_headnorm_kvwrite_kernel(const T* __restrict__ u, int64_t u_stride, const fl
                              const int32_t* __restrict__ slot_mapping, const float* __restrict__ q_norm_w,
                              const float* __restrict__ k_norm_w, T* __restrict__ q_out /* [n, H*d] */,
                              T* __restrict__ k_cache /* [slots, G*d] */, T* __restrict__ v_cache /* [slots, G*dv] */,
-                             int n_tokens, int H, int G, int d, int dv, int taps, float eps) {
+                             int n_tokens, int H, int G, int d, int dv, int taps, float eps, const ConvHeadOps ops) {
+  __shared__ float rbuf[CONV_WARPS][32 * CONV_MAX_PER_LANE];
   const int lane = threadIdx.x & 31;
   const int item = blockIdx.x * CONV_WARPS + (threadIdx.x >> 5);
   const int heads = H + 2 * G;
@@ -182,21 +211,38 @@ conv_headnorm_kvwrite_kernel(const T* __restrict__ u, int64_t u_stride, const fl
         }
       }
       y[i] = acc;
-      ssq += acc * acc;
     }
   }
-  if (kind != 2) {
+  if (kind != 2 && (ops.flags & CONV_ROUND)) {
     // the projection and convolution outputs are activations: the norm reads them as stored in T
-    ssq = 0.f;
 #pragma unroll
-    for (int i = 0; i < CONV_MAX_PER_LANE; ++i) { y[i] = to_f(from_f<T>(y[i])); ssq += y[i] * y[i]; }
-    ssq = warp_sum(ssq);
-    const float inv = 1.0f / sqrtf(ssq / static_cast<float>(width) + eps);
-    const float* w = kind == 0 ? q_norm_w : k_norm_w;
+    for (int i = 0; i < CONV_MAX_PER_LANE; ++i) y[i] = to_f(from_f<T>(y[i]));
+  }
+  if (kind != 2 && ops.rot_dims > 0) {
+    float* buf = rbuf[threadIdx.x >> 5];
+    const int half = ops.rot_dims / 2;
+    const float* rt = ops.rot + static_cast<size_t>(n) * ops.rot_dims;
+#pragma unroll
+    for (int i = 0; i < CONV_MAX_PER_LANE; ++i) buf[lane + 32 * i] = y[i];
+    __syncwarp();
 #pragma unroll
     for (int i = 0; i < CONV_MAX_PER_LANE; ++i) {
       const int cc = lane + 32 * i;
-      if (cc < width) y[i] = y[i] * inv * w[cc];
+      if (cc < half) y[i] = y[i] * rt[cc] - buf[cc + half] * rt[half + cc];
+      else if (cc < ops.rot_dims) y[i] = y[i] * rt[cc - half] + buf[cc - half] * rt[cc];
+    }
+  }
+  if (kind != 2 || (ops.flags & CONV_UNIT_V)) {
+    ssq = 0.f;
+#pragma unroll
+    for (int i = 0; i < CONV_MAX_PER_LANE; ++i) ssq += y[i] * y[i];
+    ssq = warp_sum(ssq);
+    const float inv = 1.0f / sqrtf(ssq / static_cast<float>(width) + eps);
+    const float* w = kind == 0 ? q_norm_w : kind == 1 ? k_norm_w : nullptr;
+#pragma unroll
+    for (int i = 0; i < CONV_MAX_PER_LANE; ++i) {
+      const int cc = lane + 32 * i;
+      if (cc < width) y[i] = y[i] * inv * (w != nullptr ? w[cc] : 1.f);
     }
   }
   T* dst = kind == 0 ? q_out + static_cast<size_t>(n) * H * d + head * d
@@ -226,7 +272,7 @@ constexpr int CONV4_CHUNKS = 2;            // head sizes up to 256
 constexpr int CONV4_TOKENS = 8;            // consecutive rows of the step per warp: the taps' weights are loaded once for all
 
 // One warp per (block of CONV4_TOKENS rows, head slice).  The lane keeps the taps of its four channels in registers.
-template <typename T, int TAPS, int NCH>
+template <typename T, int TAPS, int NCH, bool ROT>
 __global__ void __launch_bounds__(CONV_WARPS * 32)
 conv_headnorm_kvwrite_vec4_kernel(const T* __restrict__ u, int64_t u_stride, const float* __restrict__ conv_w,
                                   const T* __restrict__ state, const int32_t* __restrict__ tok_seq,
@@ -234,7 +280,9 @@ conv_headnorm_kvwrite_vec4_kernel(const T* __restrict__ u, int64_t u_stride, con
                                   const int32_t* __restrict__ seq_pos0, const int32_t* __restrict__ seq_slot,
                                   const int32_t* __restrict__ slot_mapping, const float* __restrict__ q_norm_w,
                                   const float* __restrict__ k_norm_w, T* __restrict__ q_out, T* __restrict__ k_cache,
-                                  T* __restrict__ v_cache, int n_tokens, int H, int G, int d, int dv, float eps) {
+                                  T* __restrict__ v_cache, int n_tokens, int H, int G, int d, int dv, float eps,
+                                  const ConvHeadOps ops) {
+  __shared__ __align__(16) float rbuf[CONV_WARPS][ROT ? 128 * NCH : 4];
   const int lane = threadIdx.x & 31;
   const int item = blockIdx.x * CONV_WARPS + (threadIdx.x >> 5);
   const int heads = H + 2 * G;
@@ -254,7 +302,7 @@ conv_headnorm_kvwrite_vec4_kernel(const T* __restrict__ u, int64_t u_stride, con
     const int cc = (lane + 32 * i) * 4;
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      g4[i][e] = 0.f;
+      g4[i][e] = 1.f;
 #pragma unroll
       for (int j = 0; j < TAPS; ++j) w[i][e][j] = 0.f;
     }
@@ -270,7 +318,7 @@ conv_headnorm_kvwrite_vec4_kernel(const T* __restrict__ u, int64_t u_stride, con
       for (int e = 0; e < 4; ++e)
 #pragma unroll
         for (int j = 0; j < TAPS; ++j) w[i][e][j] = flat[e * TAPS + j];
-      if (kind != 2) {
+      if (kind != 2 && q_norm_w != nullptr) {
         const float4 r = *reinterpret_cast<const float4*>((kind == 0 ? q_norm_w : k_norm_w) + cc);
         g4[i][0] = r.x; g4[i][1] = r.y; g4[i][2] = r.z; g4[i][3] = r.w;
       }
@@ -286,14 +334,45 @@ conv_headnorm_kvwrite_vec4_kernel(const T* __restrict__ u, int64_t u_stride, con
       m_pos0 = seq_pos0[b]; m_start = seq_start[b]; m_sslot = seq_slot[b];
     }
   }
-  // norm of a q / k head (the convolution's output rounded to T first), then the row's destination
+  // rotation and norm of a head (see ConvHeadOps), then the row's destination
   auto finish = [&](float (&y)[NCH][4], int n, int slot) {
-    if (kind != 2) {
+    if (kind != 2 && (ops.flags & CONV_ROUND)) {
+#pragma unroll
+      for (int i = 0; i < NCH; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y[i][e] = to_f(from_f<T>(y[i][e]));
+    }
+    if constexpr (ROT) {
+      if (kind != 2) {                                   // rot_dims / 2 is a multiple of four: partners are whole quads
+        float* buf = rbuf[threadIdx.x >> 5];
+        const int half = ops.rot_dims / 2;
+        const float* rt = ops.rot + static_cast<size_t>(n) * ops.rot_dims;
+        __syncwarp();                                    // the previous row's reads
+#pragma unroll
+        for (int i = 0; i < NCH; ++i) Vec4<float>::store(buf + (lane + 32 * i) * 4, y[i]);
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < NCH; ++i) {
+          const int cc = (lane + 32 * i) * 4;
+          if (cc < ops.rot_dims) {
+            const bool first = cc < half;
+            const int c1 = first ? cc : cc - half;
+            float cs[4], sn[4], pr[4];
+            Vec4<float>::load(rt + c1, cs);
+            Vec4<float>::load(rt + half + c1, sn);
+            Vec4<float>::load(buf + (first ? cc + half : c1), pr);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) y[i][e] = first ? y[i][e] * cs[e] - pr[e] * sn[e] : y[i][e] * cs[e] + pr[e] * sn[e];
+          }
+        }
+      }
+    }
+    if (kind != 2 || (ops.flags & CONV_UNIT_V)) {
       float ssq = 0.f;
 #pragma unroll
       for (int i = 0; i < NCH; ++i)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) { y[i][e] = to_f(from_f<T>(y[i][e])); ssq += y[i][e] * y[i][e]; }
+        for (int e = 0; e < 4; ++e) ssq += y[i][e] * y[i][e];
       ssq = warp_sum(ssq);
       const float inv = 1.0f / sqrtf(ssq / static_cast<float>(width) + eps);
 #pragma unroll
@@ -525,10 +604,11 @@ static void launch_conv(bool vec4, int grid, cudaStream_t st, const void* u, int
                         const int32_t* tok_seq, const int32_t* positions, const int32_t* seq_start, const int32_t* seq_pos0,
                         const int32_t* seq_len, const int32_t* seq_slot, const int32_t* slot_mapping, const float* q_norm_w,
                         const float* k_norm_w, void* q_out, void* k_cache, void* v_cache, int n_tokens, int n_seqs, int H, int G, int d,
-                        int dv, int taps, float eps, int C) {
-#define CONV4_GO_N(TP, NCH) conv_headnorm_kvwrite_vec4_kernel<T, TP, NCH><<<grid, CONV_WARPS * 32, 0, st>>>(static_cast<const T*>(u), u_stride, conv_w, \
+                        int dv, int taps, float eps, int C, const ConvHeadOps& ops) {
+#define CONV4_GO_R(TP, NCH, ROT) conv_headnorm_kvwrite_vec4_kernel<T, TP, NCH, ROT><<<grid, CONV_WARPS * 32, 0, st>>>(static_cast<const T*>(u), u_stride, conv_w, \
       static_cast<const T*>(state), tok_seq, positions, seq_start, seq_pos0, seq_slot, slot_mapping, q_norm_w, k_norm_w, \
-      static_cast<T*>(q_out), static_cast<T*>(k_cache), static_cast<T*>(v_cache), n_tokens, H, G, d, dv, eps)
+      static_cast<T*>(q_out), static_cast<T*>(k_cache), static_cast<T*>(v_cache), n_tokens, H, G, d, dv, eps, ops)
+#define CONV4_GO_N(TP, NCH) do { if (ops.rot_dims > 0) CONV4_GO_R(TP, NCH, true); else CONV4_GO_R(TP, NCH, false); } while (0)
 #define CONV4_GO(TP) do { if (d <= 128 && dv <= 128) CONV4_GO_N(TP, 1); else CONV4_GO_N(TP, 2); } while (0)
   if (vec4) grid = ((n_tokens + CONV4_TOKENS - 1) / CONV4_TOKENS * (H + 2 * G) + CONV_WARPS - 1) / CONV_WARPS;
   if (vec4 && taps == 4) CONV4_GO(4);
@@ -538,9 +618,10 @@ static void launch_conv(bool vec4, int grid, cudaStream_t st, const void* u, int
   else
     conv_headnorm_kvwrite_kernel<T><<<grid, CONV_WARPS * 32, 0, st>>>(static_cast<const T*>(u), u_stride, conv_w, static_cast<const T*>(state),
         tok_seq, positions, seq_start, seq_pos0, seq_slot, slot_mapping, q_norm_w, k_norm_w, static_cast<T*>(q_out),
-        static_cast<T*>(k_cache), static_cast<T*>(v_cache), n_tokens, H, G, d, dv, taps, eps);
+        static_cast<T*>(k_cache), static_cast<T*>(v_cache), n_tokens, H, G, d, dv, taps, eps, ops);
 #undef CONV4_GO
 #undef CONV4_GO_N
+#undef CONV4_GO_R
   if (taps > 1)
     conv_state_update_kernel<T><<<dim3((C + 127) / 128, n_seqs), 128, 0, st>>>(static_cast<const T*>(u), u_stride, static_cast<T*>(state),
         seq_start, seq_pos0, seq_len, seq_slot, n_seqs, C, taps);
@@ -621,22 +702,38 @@ extern "C" int b2tts_relu_sq(void* y, int64_t n, int dtype, void* stream) {
   return B2TTS_OK;
 }
 
+extern "C" int b2tts_rotary_table(const int32_t* positions, const float* freq, float* table, int n, int half, void* stream) {
+  using namespace b2;
+  B2_REQUIRE(n >= 0 && half >= 0, B2TTS_EINVAL, "rotary_table: n=%d half=%d", n, half);
+  if (n == 0 || half == 0) return B2TTS_OK;
+  B2_REQUIRE(positions && freq && table, B2TTS_EINVAL, "rotary_table: null pointer");
+  const size_t total = static_cast<size_t>(n) * half;
+  rotary_table_kernel<<<static_cast<unsigned>((total + 255) / 256), 256, 0, static_cast<cudaStream_t>(stream)>>>(positions, freq, table, n, half);
+  B2_CHECK_LAUNCH("rotary_table");
+  return B2TTS_OK;
+}
+
 extern "C" int b2tts_conv_headnorm_kvwrite(const void* u, int64_t u_stride, const float* conv_w, void* state,
                                            const int32_t* tok_seq, const int32_t* positions, const int32_t* seq_start,
                                            const int32_t* seq_pos0, const int32_t* seq_len, const int32_t* seq_slot,
                                            const int32_t* slot_mapping, const float* q_norm_w, const float* k_norm_w,
                                            void* q_out, void* k_cache, void* v_cache, int n_tokens, int n_seqs, int heads,
-                                           int kv_heads, int dim, int vdim, int taps, float eps, int dtype, void* stream) {
+                                           int kv_heads, int dim, int vdim, int taps, float eps, const float* rot, int rot_dims,
+                                           int flags, int dtype, void* stream) {
   using namespace b2;
   B2_REQUIRE(n_tokens >= 0 && n_seqs >= 0 && heads > 0 && kv_heads > 0 && dim > 0 && vdim > 0, B2TTS_EINVAL,
              "conv_headnorm_kvwrite: bad sizes");
+  B2_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dim && (rot_dims == 0 || rot), B2TTS_EINVAL,
+             "conv_headnorm_kvwrite: %d rotated of %d coordinates", rot_dims, dim);
+  B2_REQUIRE((flags & ~(CONV_ROUND | CONV_UNIT_V)) == 0 && (q_norm_w == nullptr) == (k_norm_w == nullptr), B2TTS_EINVAL,
+             "conv_headnorm_kvwrite: flags %d, or a norm weight for only one of q and k", flags);
   B2_REQUIRE(taps >= 1 && taps <= CONV_MAX_TAPS, B2TTS_EUNSUPPORTED, "conv_headnorm_kvwrite: taps %d not in 1..%d", taps, CONV_MAX_TAPS);
   B2_REQUIRE(dim <= 32 * CONV_MAX_PER_LANE && vdim <= 32 * CONV_MAX_PER_LANE, B2TTS_EUNSUPPORTED,
              "conv_headnorm_kvwrite: head size above %d", 32 * CONV_MAX_PER_LANE);
   B2_REQUIRE(LM_DTYPE_OK(dtype), B2TTS_EINVAL, "conv_headnorm_kvwrite: dtype %d", dtype);
   if (n_tokens == 0 || n_seqs == 0) return B2TTS_OK;
   B2_REQUIRE(u && conv_w && (state || taps == 1) && tok_seq && positions && seq_start && seq_pos0 && seq_len && seq_slot &&
-             slot_mapping && q_norm_w && k_norm_w && q_out && k_cache && v_cache, B2TTS_EINVAL, "conv_headnorm_kvwrite: null pointer");
+             slot_mapping && q_out && k_cache && v_cache, B2TTS_EINVAL, "conv_headnorm_kvwrite: null pointer");
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int items = n_tokens * (heads + 2 * kv_heads);
   const int grid = (items + CONV_WARPS - 1) / CONV_WARPS;
@@ -644,13 +741,15 @@ extern "C" int b2tts_conv_headnorm_kvwrite(const void* u, int64_t u_stride, cons
   // four channels per lane when every head slice and row starts on a 16-byte (float) / 8-byte (bf16) boundary
   const bool vec4 = dim % 4 == 0 && vdim % 4 == 0 && u_stride % 4 == 0 && dim <= 128 * CONV4_CHUNKS && vdim <= 128 * CONV4_CHUNKS &&
                     (taps == 1 || taps == 2 || taps == 3 || taps == 4) && aligned16(u) && aligned16(q_out) && aligned16(k_cache) &&
-                    aligned16(v_cache) && aligned16(conv_w) && aligned16(q_norm_w) && aligned16(k_norm_w) && (taps == 1 || aligned16(state));
+                    aligned16(v_cache) && aligned16(conv_w) && (!q_norm_w || (aligned16(q_norm_w) && aligned16(k_norm_w))) && (taps == 1 || aligned16(state)) &&
+                    (rot_dims == 0 || (rot_dims % 8 == 0 && aligned16(rot)));
+  const ConvHeadOps ops{rot, rot_dims, flags};
   if (dtype == B2TTS_DTYPE_BF16)
     launch_conv<__nv_bfloat16>(vec4, grid, st, u, u_stride, conv_w, state, tok_seq, positions, seq_start, seq_pos0, seq_len, seq_slot,
-                               slot_mapping, q_norm_w, k_norm_w, q_out, k_cache, v_cache, n_tokens, n_seqs, heads, kv_heads, dim, vdim, taps, eps, C);
+                               slot_mapping, q_norm_w, k_norm_w, q_out, k_cache, v_cache, n_tokens, n_seqs, heads, kv_heads, dim, vdim, taps, eps, C, ops);
   else
     launch_conv<float>(vec4, grid, st, u, u_stride, conv_w, state, tok_seq, positions, seq_start, seq_pos0, seq_len, seq_slot,
-                       slot_mapping, q_norm_w, k_norm_w, q_out, k_cache, v_cache, n_tokens, n_seqs, heads, kv_heads, dim, vdim, taps, eps, C);
+                       slot_mapping, q_norm_w, k_norm_w, q_out, k_cache, v_cache, n_tokens, n_seqs, heads, kv_heads, dim, vdim, taps, eps, C, ops);
   B2_CHECK_LAUNCH("conv_headnorm_kvwrite");
   return B2TTS_OK;
 }

@@ -5,8 +5,10 @@
 //                    with log gates i, f and the running maximum m = max(f + m, i), a = exp(f + m_old - m), b = exp(i - m)
 //   delta rule       S <- g S;  u = beta (v - S^T k);  S <- S + k u^T      o = S^T q
 //   gated linear     S <- diag(alpha) S + k v^T                            o = S^T q      (a decay per key channel and token)
+//   retention        S <- decay_h S + k v^T                                o = S^T q      (a fixed decay per head; retention.cu
+//                                                                                         has its tensor-core and one-token kernels)
 //
-// All three update every value column of S independently.  A column is shared by RS = ceil(key size / 32) lanes of one
+// All of them update every value column of S independently.  A column is shared by RS = ceil(key size / 32) lanes of one
 // warp, each keeping 32 rows of it in registers for the whole portion; sums over the rows (the read-out, the delta rule's
 // S^T k, the unit norms) are butterfly shuffles over those lanes.  The per-token vectors (k, q or B, C) are staged in
 // shared memory one element per thread (one barrier per token), their loads run four tokens ahead through registers, and
@@ -37,6 +39,8 @@ struct ScanArgs {
   const void* q; int64_t ldq;             // query-like vectors, same layout
   const void* v; int64_t ldv;             // values: (row, head h, c) at v[row * ldv + h * dv + c]
   const float* coef;                      // [rows, H, 3] per-token scalars, see scan_kernel (SCAN_GATED: unused)
+  const float* head_decay;                // [H] or null: coef = (head_decay[h], 1, 1) for every token (coef itself is then unused)
+  int rows;                               // 0: every sequence, 1: only those with more than one new token, 2: only one-token ones
   const float* decay; int64_t ldd;        // SCAN_GATED: per key channel, (row, head h, i) at decay[row * ldd + h * d + i]
   const float* skip;                      // [H] or null: out += skip[h] * value
   float* state;                           // [slots, H, d, dv]
@@ -72,7 +76,7 @@ scan_kernel(const ScanArgs a) {
   __shared__ __align__(16) float vec[2][SCAN_DEPTH][NV][DP];  // [buffer][token of the group][k | q | decay][row]
   const int b = blockIdx.z, h = blockIdx.y;
   const int len = a.seq_len[b];
-  if (len <= 0) return;
+  if (len <= 0 || (a.rows == 1 && len == 1) || (a.rows == 2 && len > 1)) return;
   const int d = a.d, dv = a.dv, H = a.H;
   const int g = h / (H / a.G);
   const int start = a.seq_start[b], pos0 = a.seq_pos0[b];
@@ -95,6 +99,7 @@ scan_kernel(const ScanArgs a) {
   const float* dp = KIND == SCAN_GATED ? a.decay + static_cast<size_t>(start) * a.ldd + h * d + tid : nullptr;
   float* op = a.out + static_cast<size_t>(start) * H * dv + h * dv + col;
   const float skip = a.skip != nullptr ? a.skip[h] : 0.f;
+  const float fixed = a.head_decay != nullptr ? a.head_decay[h] : 0.f;
 
   // the loaded values stay as they came (type T) until their token is staged: converting them at once would make the
   // thread wait for the load, four tokens early
@@ -109,6 +114,8 @@ scan_kernel(const ScanArgs a) {
       if (live) rv[u] = vp[static_cast<size_t>(t) * a.ldv];
       if constexpr (KIND == SCAN_GATED) {
         if (mine) rd[u] = dp[static_cast<size_t>(t) * a.ldd];
+      } else if (a.head_decay != nullptr) {
+        rc[u][0] = fixed; rc[u][1] = 1.f; rc[u][2] = 1.f;
       } else {
         const float* c = cp + static_cast<size_t>(t) * H * 3;
         rc[u][0] = c[0]; rc[u][1] = c[1]; rc[u][2] = c[2];
@@ -470,5 +477,25 @@ extern "C" int b2tts_gated_linear_scan(const void* q, int64_t ldq, const void* k
                                            : launch_scan<float, SCAN_GATED>(a, n_seqs, st, "gated_linear_scan");
   if (rc != B2TTS_OK) return rc;
   B2_CHECK_LAUNCH("gated_linear_scan");
+  return B2TTS_OK;
+}
+
+extern "C" int b2tts_fixed_decay_scan(const float* q, int64_t ldq, const float* k, int64_t ldk, const float* v, int64_t ldv,
+                                      const float* head_decay, float* state, float* out, const int32_t* seq_start,
+                                      const int32_t* seq_pos0, const int32_t* seq_len, const int32_t* seq_slot, int n_tokens,
+                                      int n_seqs, int heads, int dim, int vdim, int rows, void* stream) {
+  const int dtype = B2TTS_DTYPE_F32;
+  SCAN_COMMON_CHECKS("fixed_decay_scan");
+  if (n_tokens <= 0) return B2TTS_OK;
+  B2_REQUIRE(q && k && v && head_decay && rows >= 0 && rows <= 2, B2TTS_EINVAL, "fixed_decay_scan: null pointer or rows %d", rows);
+  ScanArgs a{};
+  a.q = q; a.ldq = ldq; a.k = k; a.ldk = ldk; a.v = v; a.ldv = ldv;
+  a.head_decay = head_decay; a.rows = rows;
+  a.state = state; a.out = out;
+  a.seq_start = seq_start; a.seq_pos0 = seq_pos0; a.seq_len = seq_len; a.seq_slot = seq_slot;
+  a.H = heads; a.G = heads; a.d = dim; a.dv = vdim; a.qscale = 1.f; a.divide = 0;
+  const int rc = launch_scan<float, SCAN_LINEAR>(a, n_seqs, static_cast<cudaStream_t>(stream), "fixed_decay_scan");
+  if (rc != B2TTS_OK) return rc;
+  B2_CHECK_LAUNCH("fixed_decay_scan");
   return B2TTS_OK;
 }

@@ -98,3 +98,37 @@ class StreamRMSNorm(nn.Module):
 
     def forward(self, xs: torch.Tensor, dtype: torch.dtype, rows: torch.Tensor | None = None) -> torch.Tensor:
         return nat.stream_gather_norm(xs, rows, None, self.weight, self.eps, dtype)
+
+
+class OffsetRMSNorm(nn.Module):
+    """RMS norm whose checkpoint weight is the distance from one: y = x / sqrt(mean(x^2) + eps) * (1 + w), over a 32-bit
+    residual stream.  ``weight`` keeps the sum 1 + w in float (``from_stored``).  In a model the norm rides in the residual
+    update in front of it (``GatedResidual``); ``forward`` is the stand-alone form on gathered rows (the final norm)."""
+
+    def __init__(self, width: int, eps: float = 1e-6):
+        super().__init__()
+        self.eps = eps
+        self.weight = nn.Parameter(torch.ones(width, dtype=torch.float32), requires_grad=False)
+
+    @staticmethod
+    def from_stored(w: torch.Tensor) -> torch.Tensor:
+        return 1.0 + w.to(torch.float32)
+
+    def forward(self, x: torch.Tensor, dtype: torch.dtype, rows: torch.Tensor | None = None) -> torch.Tensor:
+        return nat.gather_group_norm(x, rows, self.weight, 1, self.eps, dtype)
+
+
+class GatedResidual(nn.Module):
+    """Gate of a sublayer's result on its way into a 32-bit residual stream: x += sigmoid(z + b) * y with z = W h, h the
+    sublayer's input (W rides in a projection of the sublayer; the bias is kept here in float).  ``forward`` updates x in
+    place and, in the same launch, adds what comes in front of the next sublayer (``table`` rows ``index``, a vector
+    ``add``) and returns its input ``nxt(x)`` (None without ``nxt``)."""
+
+    def __init__(self, width: int):
+        super().__init__()
+        self.bias = nn.Parameter(torch.zeros(width, dtype=torch.float32), requires_grad=False)
+
+    def forward(self, x: torch.Tensor, y: torch.Tensor, z: torch.Tensor, nxt: OffsetRMSNorm | None = None, *, table=None, index=None,
+                add=None) -> torch.Tensor | None:
+        return nat.gated_residual(x, y=y, z=z, zb=self.bias, table=table, index=index, add=add, w=nxt.weight if nxt is not None else None,
+                                  eps=nxt.eps if nxt is not None else 0.0)

@@ -159,6 +159,15 @@ def linear_relu_sq(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
     return nat.relu_sq_(linear(x, weight))
 
 
+def linear_gelu_mul(x: torch.Tensor, gate_up_weight: torch.Tensor) -> torch.Tensor:
+    """gelu_tanh(x Wg^T) * (x Wu^T) over the merged [gate; up] weight, with the activation in the GEMM epilogue on the
+    native path; the library GEMM followed by the gated product elsewhere (long prompts, float32)."""
+    m, n = x.shape[0], gate_up_weight.shape[0]
+    if x.dtype == torch.bfloat16 and native_ok(m, n, x.shape[1]):
+        return nat.gemm_bf16(x, packed_weight(gate_up_weight, nat.PACK_GATE_UP), n, epilogue=nat.GEMM_GELU_MUL, pdl=PDL)
+    return nat.gelu_mul(linear(x, gate_up_weight))
+
+
 def per_head_linear(x: torch.Tensor, weight: torch.Tensor, transpose_weight: bool = False) -> torch.Tensor:
     """One small projection per head, all heads in one strided-batched library GEMM (cuBLAS through ``torch.bmm``):
     x [heads, n, k] (any strides) and weight [heads, k, m] (or [heads, m, k] with ``transpose_weight``) -> [heads, n, m]."""
@@ -203,11 +212,17 @@ class RowParallelLinear(LinearBase):
 
 class MergedColumnParallelLinear(ColumnParallelLinear):
     """Several column-parallel projections sharing one input, stored as one weight so that one GEMM
-    serves them (gate|up, q|k|v).  ``weight_loader(param, w, shard_id)`` fills one shard."""
+    serves them (gate|up, q|k|v).  ``weight_loader(param, w, shard_id)`` fills one shard.  ``pad_to``: the weight gets
+    rows of zeros behind the last shard up to a multiple of it, so that odd shards (a number per head) leave the output
+    rows on vector boundaries and the product on the native kernel's tiles."""
 
-    def __init__(self, input_size: int, output_sizes: list[int], bias: bool = False):
+    def __init__(self, input_size: int, output_sizes: list[int], bias: bool = False, pad_to: int = 1):
         self.output_sizes = list(output_sizes)
-        super().__init__(input_size, sum(output_sizes), bias)
+        n = sum(output_sizes)
+        super().__init__(input_size, -(-n // pad_to) * pad_to, bias)
+        if self.weight.shape[0] > n:
+            with torch.no_grad():
+                self.weight[n:].zero_()
 
     def weight_loader(self, param: nn.Parameter, loaded_weight: torch.Tensor, loaded_shard_id: int = None):
         with torch.no_grad():

@@ -169,3 +169,37 @@ class GatedLinearAttention(nn.Module):
         out = torch.empty(n, hv, dtype=u.dtype, device=u.device)
         nat.gated_group_norm(o, cut("g", hv), self.norm, m.heads, nat.GATE_SILU, False, self.eps, out)
         return out
+
+
+class Retention(nn.Module):
+    """Retention: S <- decay_h S + k v^T, o = S^T q per head with a fixed decay per head; q and k rotated (``rotary``: a
+    ``HalfRotaryTable`` or None), k scaled by dim^(-1/2); each head's read-out divided by its root mean square, then
+    multiplied by silu(W_g h).  A step of single tokens is one launch; prompt portions run in chunks on the tensor cores in
+    bf16 where the sizes allow, and token by token otherwise."""
+
+    def __init__(self, spec, eps: float, rotary=None):
+        super().__init__()
+        self.spec, self.eps, self.rotary = spec, eps, rotary
+        self.register_buffer("decay", torch.tensor(spec.decay, dtype=torch.float64).to(torch.float32), persistent=False)
+        self.path = nat.RETENTION_AUTO
+        self.S = None
+
+    def proj_parts(self):
+        m = self.spec
+        return [("q", m.heads * m.dim), ("k", m.heads * m.dim), ("v", m.heads * m.vdim), ("g", m.heads * m.vdim)]
+
+    def state_plan(self):
+        m = self.spec
+        return [((m.heads, m.dim, m.vdim), torch.float32)]
+
+    def bind(self, state):
+        (self.S,) = state
+
+    def forward(self, u: torch.Tensor, cols: dict) -> torch.Tensor:
+        m, lay = self.spec, get_context().step_layout
+        hd, hv = m.heads * m.dim, m.heads * m.vdim
+        cut = lambda name, w: u[:, cols[name]:cols[name] + w]
+        out = torch.empty(u.shape[0], hv, dtype=u.dtype, device=u.device)
+        nat.retention(cut("q", hd), cut("k", hd), cut("v", hv), self.rotary.table if self.rotary is not None else None, self.decay,
+                      m.dim ** -0.5, self.S, cut("g", hv), out, lay, m.heads, m.dim, m.vdim, self.eps, self.path)
+        return out

@@ -114,3 +114,15 @@ class HalfRotary(nn.Module):
         self.register_buffer("freq", f.to(torch.float32), persistent=False)
 
     interleaved = False
+
+
+class HalfRotaryTable(HalfRotary):
+    """The same rotation for kernels that read cosines and sines from a table: ``fill`` computes the table of a step's
+    positions once ([n, dims]: cosines, then sines), every layer with the same frequencies then shares ``table``."""
+
+    def __init__(self, dims: int, base: float):
+        super().__init__(dims, base)
+        self.table = None
+
+    def fill(self, positions: torch.Tensor) -> None:
+        self.table = nat.rotary_table(positions, self.freq)

@@ -32,6 +32,30 @@ class ShortConvQKV(nn.Module):
         return q
 
 
+class ShortConvRotaryQKV(nn.Module):
+    """The same fusion for heads that are rotated and unit-normed: convolution -> rotation of q and k (``rotary``: a
+    ``HalfRotaryTable`` or None) -> q, k and v heads divided by their root mean square, without weights -> k, v to their cache
+    slots, all in float from the projection on."""
+
+    def __init__(self, heads: int, kv_heads: int, dim: int, vdim: int, taps: int, eps: float, rotary=None):
+        super().__init__()
+        self.heads, self.kv_heads, self.dim, self.vdim, self.taps, self.eps, self.rotary = heads, kv_heads, dim, vdim, taps, eps, rotary
+        self.channels = heads * dim + kv_heads * (dim + vdim)
+        self.weight = nn.Parameter(torch.zeros(self.channels, taps, dtype=torch.float32), requires_grad=False)
+        self.state = None                      # [slots, max(taps - 1, 1), channels], bound by the model runner
+
+    def state_plan(self):
+        return ((max(self.taps - 1, 1), self.channels), None)
+
+    def forward(self, u: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor) -> torch.Tensor:
+        """u [n, >= channels], its first columns q | k | v -> q [n, heads * dim]."""
+        q = torch.empty(u.shape[0], self.heads * self.dim, dtype=u.dtype, device=u.device)
+        nat.conv_headnorm_kvwrite(u, self.weight, self.state, get_context().step_layout, None, None, q, k_cache, v_cache, self.heads,
+                                  self.kv_heads, self.dim, self.vdim, self.taps, self.eps,
+                                  rot=self.rotary.table if self.rotary is not None else None, flags=nat.CONV_UNIT_V)
+        return q
+
+
 F32 = dict(dtype=torch.float32)
 
 
