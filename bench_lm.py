@@ -68,7 +68,8 @@ def bench_bokenex(s: dict, moe: bool, device: str, design: str = "bokenex") -> d
     import torch
     from nano_qwen3tts_vllm_b200.engine.llm_engine.lm_engine import CausalLMEngine
     from nano_qwen3tts_vllm_b200.sampling_params import SamplingParams
-    cfg = {"bokenex": bokenex_config, "ridevik": ridevik_config, "tibivik": tibivik_config, "teberax": teberax_config}[design](s, moe)
+    cfg = {"bokenex": bokenex_config, "ridevik": ridevik_config, "tibivik": tibivik_config, "teberax": teberax_config,
+           "zekivik": zekivik_config}[design](s, moe)
     pages = DECODE_SEQS * ((DECODE_CTX + 64 + PAGE - 1) // PAGE) + PREFILL_SEQS * (PREFILL_LEN // PAGE + 1)
     eng = CausalLMEngine(cfg, state_dict="random:7", kvcache_block_size=PAGE, num_kvcache_blocks=pages,
                          max_num_seqs=DECODE_SEQS + PREFILL_SEQS, max_model_len=4096, max_num_batched_tokens=16384,
@@ -753,6 +754,151 @@ def main_teberax(device: str = "cuda:0") -> dict:
         torch.cuda.empty_cache()
     out["kernels"] = bench_teberax_kernels(device)
     out["like_kernels"] = bench_hybrid_kernels(device)
+    out["seconds"] = round(time.time() - t0, 1)
+    return out
+
+
+def zekivik_config(s: dict, moe: bool = False):
+    """Layers of a real model's shape at the size's width: causal convolved attention of the size's head layout alternating
+    with retention of as many heads of 128 x 128, every layer with a GELU-gated feed-forward of three matrices of the talker's
+    parameter count; no looped range (as many layer runs as the model it is compared with)."""
+    from nano_qwen3tts_vllm_b200.config import ZekivikConfig
+    d, H, G = s["dim"], s["heads"], s["kv_heads"]
+    mlp = {"kind": "dense", "ff": s["inter"]}
+    rot = {"dims": d, "base": 1e6}
+    att = {"type": "attention", "mlp": mlp,
+           "mixer": {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "conv": TAPS, "scale": d ** -0.5, "rot": rot}}
+    ret = {"type": "retention", "mlp": mlp,
+           "mixer": {"heads": H, "dim": d, "vdim": d, "decay": [1 - 2.0 ** (-5 - 6 * i / (H - 1)) for i in range(H)], "rot": rot}}
+    return ZekivikConfig.from_dict({"architecture": "Zekivik", "vocab": 3072, "width": s["width"], "norm": {"eps": 1e-6},
+                                    "layers": [att, ret, att, ret][:LAYERS]})
+
+
+def bench_zekivik_kernels(device: str) -> dict:
+    """The kernels Zekivik added or extended at the w2048 layer shapes, each after an L2 flush, with the fraction of the
+    measured roofline; the like kernels come from ``bench_teberax_kernels`` and ``bench_kernels`` in the same run."""
+    import torch
+    import nano_qwen3tts_vllm_b200._native as nat
+    from nano_qwen3tts_vllm_b200.layers.linear import linear, linear_gelu_mul
+    from nano_qwen3tts_vllm_b200.layers.rotary_embedding import HalfRotaryTable
+    hbm, tflops, how = _peaks()
+    dev = torch.device(device)
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    BF = torch.bfloat16
+
+    def timed(fn, iters=5):
+        for _ in range(3):
+            fn()
+        ts = []
+        for _ in range(iters):
+            flush.zero_()
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            fn()
+            b.record()
+            torch.cuda.synchronize()
+            ts.append(a.elapsed_time(b))
+        return sorted(ts)[len(ts) // 2]
+
+    class Lay:
+        pass
+
+    def layout(n_seqs, cached, new, pages_per_seq):
+        lay = Lay()
+        i32 = dict(dtype=torch.int32, device=dev)
+        lay.n_seqs, lay.max_new, lay.n_tokens = n_seqs, new, n_seqs * new
+        lay.seq_start = torch.arange(n_seqs, **i32) * new
+        lay.seq_pos0 = torch.full((n_seqs,), cached, **i32)
+        lay.seq_len = torch.full((n_seqs,), new, **i32)
+        lay.seq_slot = torch.arange(n_seqs, **i32)
+        lay.block_tables = torch.arange(n_seqs * pages_per_seq, **i32).view(n_seqs, pages_per_seq).contiguous()
+        lay.positions = (torch.arange(new, **i32) + cached).repeat(n_seqs)
+        lay.tok_seq = torch.arange(n_seqs, **i32).repeat_interleave(new)
+        lay.slot_mapping = (lay.tok_seq * pages_per_seq * PAGE + lay.positions).to(torch.int32)
+        return lay
+
+    def entry(ms, bytes_=None, flops=None):
+        e = {"us": round(ms * 1e3, 1)}
+        if bytes_ is not None:
+            e["gbs"] = round(bytes_ / ms / 1e6, 1)
+            e["frac_hbm"] = round(bytes_ / ms / 1e6 / hbm, 3)
+        if flops is not None:
+            e["tflops"] = round(flops / ms / 1e9, 1)
+            e["frac_tensor"] = round(flops / ms / 1e9 / tflops, 4)
+        return e
+
+    H, G, d, D, ff = 16, 8, 128, 2048, 6144
+    res = {"peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "source": how}}
+    pps = (DECODE_CTX + PAGE) // PAGE + 1
+    dlay, play = layout(DECODE_SEQS, DECODE_CTX, 1, pps), layout(PREFILL_SEQS, 0, PREFILL_LEN, PREFILL_LEN // PAGE)
+    n = PREFILL_SEQS * PREFILL_LEN
+    rot = HalfRotaryTable(d, 1e6).to(dev)
+    tables = {id(l): nat.rotary_table(l.positions, rot.freq) for l in (dlay, play)}
+    res["rotary_table 8192 tokens"] = entry(timed(lambda: nat.rotary_table(play.positions, rot.freq)), bytes_=n * d * 4)
+    # ---- attention: causal, ordinary softmax, a gate per head
+    kc = torch.randn(DECODE_SEQS * pps, PAGE, G * d, device=dev).to(BF)
+    vc = torch.randn(DECODE_SEQS * pps, PAGE, G * d, device=dev).to(BF)
+
+    def attn(lay):
+        q = torch.randn(lay.n_tokens, H * d, device=dev).to(BF)
+        gate = torch.randn(lay.n_tokens, H, device=dev).to(BF)
+        out = torch.empty(lay.n_tokens, H * d, dtype=BF, device=dev)
+        return lambda: nat.sink_attn(q, kc, vc, out, lay, None, gate, H, G, d, d, PAGE, nat.MASK_WINDOW, 0, d ** -0.5)
+
+    pairs = PREFILL_SEQS * sum(i + 1 for i in range(PREFILL_LEN))
+    res["sink_attn prefill 4x2048 causal, head gate"] = entry(timed(attn(play), iters=3), flops=pairs * H * 2 * d * 2)
+    res["sink_attn decode 64x1100 causal, head gate"] = entry(timed(attn(dlay)), bytes_=DECODE_SEQS * (DECODE_CTX + 1) * G * d * 2 * 2)
+    # ---- convolution + rotation + unit norms + K/V write on the merged projection
+    C = H * d + 2 * G * d
+    for name, lay in (("8192 tokens", play), ("64 tokens", dlay)):
+        u = torch.randn(lay.n_tokens, C + D + 128, device=dev).to(BF)
+        cw = torch.randn(C, TAPS, device=dev)
+        st = torch.zeros(DECODE_SEQS, TAPS - 1, C, dtype=BF, device=dev)
+        qo = torch.empty(lay.n_tokens, H * d, dtype=BF, device=dev)
+        ms = timed(lambda: nat.conv_headnorm_kvwrite(u, cw, st, lay, None, None, qo, kc, vc, H, G, d, d, TAPS, 1e-6, rot=tables[id(lay)],
+                                                     flags=nat.CONV_UNIT_V))
+        res[f"conv_headnorm_kvwrite (rotation, unit norms) {name}"] = entry(ms, bytes_=lay.n_tokens * 2 * C * 2)
+    # ---- retention: 16 heads of 128 x 128, normed and gated
+    decay = torch.full((H,), 0.999, device=dev)
+    for name, lay in (("prefill 4x2048", play), ("decode 64", dlay)):
+        m = lay.n_tokens
+        u = torch.randn(m, 4 * H * d, device=dev).to(BF)
+        st = torch.zeros(lay.n_seqs, H, d, d, device=dev)
+        out = torch.empty(m, H * d, dtype=BF, device=dev)
+        q, k, v, gt = (u[:, i * H * d:(i + 1) * H * d] for i in range(4))
+        ms = timed(lambda: nat.retention(q, k, v, tables[id(lay)], decay, d ** -0.5, st, gt, out, lay, H, d, d, 1e-6))
+        res[f"retention {name} (16 heads, 128 x 128)"] = entry(ms, bytes_=lay.n_seqs * H * d * d * 4 * 2 + m * H * d * (4 * 2 + 2),
+                                                              flops=m * H * d * d * 6)
+    # ---- gated residual + norm; the gated product
+    x, y, z = torch.randn(n, D, device=dev), torch.randn(n, D, device=dev).to(BF), torch.randn(n, 3 * D, device=dev).to(BF)
+    zb, w = torch.zeros(D, device=dev), torch.ones(D, device=dev)
+    res["gated_residual 8192x2048"] = entry(timed(lambda: nat.gated_residual(x, y=y, z=z[:, D:2 * D], zb=zb, w=w)), bytes_=n * D * (4 * 2 + 2 * 2 + 2))
+    gu = torch.randn(n, 2 * ff, device=dev).to(BF)
+    res["gelu_mul 8192x6144"] = entry(timed(lambda: nat.gelu_mul(gu)), bytes_=n * ff * 3 * 2)
+    h = torch.randn(DECODE_SEQS, D, device=dev).to(BF)
+    wgu, win = (torch.randn(r, D, device=dev).to(BF) for r in (2 * ff, C + D + 128))
+    res["gate|up GEMM + GELU product 64x2048x12288"] = entry(timed(lambda: linear_gelu_mul(h, wgu)), bytes_=2 * ff * D * 2)
+    res["merged input GEMM 64x2048x6272"] = entry(timed(lambda: linear(h, win)), bytes_=win.numel() * 2)
+    return res
+
+
+def main_zekivik(device: str = "cuda:0") -> dict:
+    """``bench.py --lm-zekivik``: Zekivik beside Teberax (the package's closest model: causal rotary attention and a linear
+    recurrence with decays over the same engine) at equal width, head layout and layer count, then the kernels of both, and
+    Bokenex's convolution kernel, against their rooflines."""
+    import torch
+    t0 = time.time()
+    out = {"metric": "lm_prefill_decode_throughput", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic (random weights)",
+           "config": {"prefill": f"{PREFILL_SEQS}x{PREFILL_LEN} tokens per step", "decode": f"{DECODE_SEQS} sequences at context {DECODE_CTX}",
+                      "layers": LAYERS, "conv_taps": TAPS, "page": PAGE}, "sizes": {}}
+    for name, s in SIZES.items():
+        row = {"zekivik": bench_bokenex(s, False, device, "zekivik"), "teberax_dense": bench_bokenex(s, False, device, "teberax")}
+        out["sizes"][name] = row
+        torch.cuda.empty_cache()
+    out["kernels"] = bench_zekivik_kernels(device)
+    out["like_kernels"] = {**bench_teberax_kernels(device),
+                           **{k: v for k, v in bench_kernels(device).items() if k.startswith("conv_headnorm")},
+                           **{k: v for k, v in bench_hybrid_kernels(device).items() if k.startswith(("gated_group_norm", "sink_attn"))}}
     out["seconds"] = round(time.time() - t0, 1)
     return out
 

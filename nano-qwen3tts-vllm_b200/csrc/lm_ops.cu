@@ -269,10 +269,11 @@ template <> struct Vec4<__nv_bfloat16> {
   __device__ static void store(__nv_bfloat16* p, const float* f) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3])); }
 };
 constexpr int CONV4_CHUNKS = 2;            // head sizes up to 256
-constexpr int CONV4_TOKENS = 8;            // consecutive rows of the step per warp: the taps' weights are loaded once for all
+constexpr int CONV4_TOKENS = 8;            // consecutive rows of a prompt step per warp: the taps' weights are loaded once for all
 
-// One warp per (block of CONV4_TOKENS rows, head slice).  The lane keeps the taps of its four channels in registers.
-template <typename T, int TAPS, int NCH, bool ROT>
+// One warp per (block of TOK rows, head slice): TOK = CONV4_TOKENS, or 1 for steps of few rows, which then spread over more
+// warps.  The lane keeps the taps of its four channels in registers.
+template <typename T, int TAPS, int NCH, bool ROT, int TOK>
 __global__ void __launch_bounds__(CONV_WARPS * 32)
 conv_headnorm_kvwrite_vec4_kernel(const T* __restrict__ u, int64_t u_stride, const float* __restrict__ conv_w,
                                   const T* __restrict__ state, const int32_t* __restrict__ tok_seq,
@@ -282,13 +283,12 @@ conv_headnorm_kvwrite_vec4_kernel(const T* __restrict__ u, int64_t u_stride, con
                                   const float* __restrict__ k_norm_w, T* __restrict__ q_out, T* __restrict__ k_cache,
                                   T* __restrict__ v_cache, int n_tokens, int H, int G, int d, int dv, float eps,
                                   const ConvHeadOps ops) {
-  __shared__ __align__(16) float rbuf[CONV_WARPS][ROT ? 128 * NCH : 4];
   const int lane = threadIdx.x & 31;
   const int item = blockIdx.x * CONV_WARPS + (threadIdx.x >> 5);
   const int heads = H + 2 * G;
-  const int n_blocks = (n_tokens + CONV4_TOKENS - 1) / CONV4_TOKENS;
+  const int n_blocks = (n_tokens + TOK - 1) / TOK;
   if (item >= n_blocks * heads) return;
-  const int n0 = (item / heads) * CONV4_TOKENS, hs = item % heads;
+  const int n0 = (item / heads) * TOK, hs = item % heads;
   const int C = H * d + G * d + G * dv;
   int kind, head, width, c0;
   if (hs < H) { kind = 0; head = hs; width = d; c0 = head * d; }
@@ -326,7 +326,7 @@ conv_headnorm_kvwrite_vec4_kernel(const T* __restrict__ u, int64_t u_stride, con
   }
   // the rows' bookkeeping (three dependent loads each) is fetched by one lane per row, all rows at once
   int m_slot = -1, m_p = 0, m_pos0 = 0, m_start = 0, m_sslot = 0;
-  if (lane < CONV4_TOKENS && n0 + lane < n_tokens) {
+  if (lane < TOK && n0 + lane < n_tokens) {
     m_slot = slot_mapping[n0 + lane];
     if (m_slot >= 0) {
       const int b = tok_seq[n0 + lane];
@@ -334,8 +334,28 @@ conv_headnorm_kvwrite_vec4_kernel(const T* __restrict__ u, int64_t u_stride, con
       m_pos0 = seq_pos0[b]; m_start = seq_start[b]; m_sslot = seq_slot[b];
     }
   }
+  // the lane's cosines and sines for row n (ROT; rot_dims / 2 is a multiple of four: partners are whole quads)
+  struct Turn { float cs[ROT ? NCH : 1][4], sn[ROT ? NCH : 1][4]; };
+  auto turn_of = [&](int n) {
+    Turn t;
+    if constexpr (ROT) {
+      const int half = ops.rot_dims / 2;
+      const float* rt = ops.rot + static_cast<size_t>(n) * ops.rot_dims;
+#pragma unroll
+      for (int i = 0; i < NCH; ++i) {
+        const int cc = (lane + 32 * i) * 4, c1 = cc < half ? cc : cc - half;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) { t.cs[i][e] = 1.f; t.sn[i][e] = 0.f; }
+        if (kind != 2 && cc < ops.rot_dims && n < n_tokens) {
+          Vec4<float>::load(rt + c1, t.cs[i]);
+          Vec4<float>::load(rt + half + c1, t.sn[i]);
+        }
+      }
+    }
+    return t;
+  };
   // rotation and norm of a head (see ConvHeadOps), then the row's destination
-  auto finish = [&](float (&y)[NCH][4], int n, int slot) {
+  auto finish = [&](float (&y)[NCH][4], int n, int slot, const Turn& turn) {
     if (kind != 2 && (ops.flags & CONV_ROUND)) {
 #pragma unroll
       for (int i = 0; i < NCH; ++i)
@@ -343,28 +363,28 @@ conv_headnorm_kvwrite_vec4_kernel(const T* __restrict__ u, int64_t u_stride, con
         for (int e = 0; e < 4; ++e) y[i][e] = to_f(from_f<T>(y[i][e]));
     }
     if constexpr (ROT) {
-      if (kind != 2) {                                   // rot_dims / 2 is a multiple of four: partners are whole quads
-        float* buf = rbuf[threadIdx.x >> 5];
+      if (kind != 2) {
         const int half = ops.rot_dims / 2;
-        const float* rt = ops.rot + static_cast<size_t>(n) * ops.rot_dims;
-        __syncwarp();                                    // the previous row's reads
-#pragma unroll
-        for (int i = 0; i < NCH; ++i) Vec4<float>::store(buf + (lane + 32 * i) * 4, y[i]);
-        __syncwarp();
+        float r[NCH][4];
 #pragma unroll
         for (int i = 0; i < NCH; ++i) {
           const int cc = (lane + 32 * i) * 4;
-          if (cc < ops.rot_dims) {
-            const bool first = cc < half;
-            const int c1 = first ? cc : cc - half;
-            float cs[4], sn[4], pr[4];
-            Vec4<float>::load(rt + c1, cs);
-            Vec4<float>::load(rt + half + c1, sn);
-            Vec4<float>::load(buf + (first ? cc + half : c1), pr);
+          const bool first = cc < half;
+          const int c2 = cc >= ops.rot_dims ? cc : first ? cc + half : cc - half;      // the partner's channel
 #pragma unroll
-            for (int e = 0; e < 4; ++e) y[i][e] = first ? y[i][e] * cs[e] - pr[e] * sn[e] : y[i][e] * cs[e] + pr[e] * sn[e];
+          for (int e = 0; e < 4; ++e) {
+            float pr = __shfl_sync(0xffffffffu, y[0][e], (c2 >> 2) & 31);
+            if constexpr (NCH == 2) {
+              const float other = __shfl_sync(0xffffffffu, y[1][e], (c2 >> 2) & 31);
+              if (c2 >= 128) pr = other;
+            }
+            r[i][e] = y[i][e] * turn.cs[i][e] + (first ? -pr : pr) * turn.sn[i][e];
           }
         }
+#pragma unroll
+        for (int i = 0; i < NCH; ++i)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) y[i][e] = r[i][e];
       }
     }
     if (kind != 2 || (ops.flags & CONV_UNIT_V)) {
@@ -389,15 +409,15 @@ conv_headnorm_kvwrite_vec4_kernel(const T* __restrict__ u, int64_t u_stride, con
       if (cc < width) Vec4<T>::store(dst + cc, y[i]);
     }
   };
-  // The usual block of a prompt portion: CONV4_TOKENS consecutive tokens of one sequence.  Their projections and the
+  // The usual block of a prompt portion: TOK consecutive tokens of one sequence.  Their projections and the
   // taps - 1 before the first are loaded once, all loads issued before the first use; row t then reads entries t .. t + R.
   const int p0 = __shfl_sync(0xffffffffu, m_p, 0), start0 = __shfl_sync(0xffffffffu, m_start, 0);
-  const bool mine = lane >= CONV4_TOKENS || (m_slot >= 0 && m_start == start0 && m_p == p0 + lane);
+  const bool mine = lane >= TOK || (m_slot >= 0 && m_start == start0 && m_p == p0 + lane);
   if (__all_sync(0xffffffffu, mine)) {
     const int pos0 = __shfl_sync(0xffffffffu, m_pos0, 0), sslot = __shfl_sync(0xffffffffu, m_sslot, 0);
-    float uv[CONV4_TOKENS + R][NCH][4];
+    float uv[TOK + R][NCH][4];
 #pragma unroll
-    for (int k = 0; k < CONV4_TOKENS + R; ++k) {
+    for (int k = 0; k < TOK + R; ++k) {
       const int pk = p0 - R + k;
 #pragma unroll
       for (int i = 0; i < NCH; ++i) {
@@ -410,8 +430,11 @@ conv_headnorm_kvwrite_vec4_kernel(const T* __restrict__ u, int64_t u_stride, con
         }
       }
     }
+    Turn ahead = turn_of(n0);                // a row ahead of its use
 #pragma unroll
-    for (int t = 0; t < CONV4_TOKENS; ++t) {
+    for (int t = 0; t < TOK; ++t) {
+      const Turn turn = ahead;
+      if (t + 1 < TOK) ahead = turn_of(n0 + t + 1);
       float y[NCH][4];
 #pragma unroll
       for (int i = 0; i < NCH; ++i)
@@ -421,13 +444,13 @@ conv_headnorm_kvwrite_vec4_kernel(const T* __restrict__ u, int64_t u_stride, con
 #pragma unroll
           for (int j = 0; j < TAPS; ++j) y[i][e] = fmaf(w[i][e][j], uv[t + j][i][e], y[i][e]);
         }
-      finish(y, n0 + t, __shfl_sync(0xffffffffu, m_slot, t));
+      finish(y, n0 + t, __shfl_sync(0xffffffffu, m_slot, t), turn);
     }
     return;
   }
   // anything else (decoded tokens, the seam of two sequences, padding): row by row
 #pragma unroll
-  for (int t = 0; t < CONV4_TOKENS; ++t) {
+  for (int t = 0; t < TOK; ++t) {
     const int n = n0 + t;
     const int slot = __shfl_sync(0xffffffffu, m_slot, t);
     if (slot < 0) continue;                  // padding row, or past the step's last row
@@ -459,7 +482,7 @@ conv_headnorm_kvwrite_vec4_kernel(const T* __restrict__ u, int64_t u_stride, con
         }
       }
     }
-    finish(y, n, slot);
+    finish(y, n, slot, turn_of(n));
   }
 }
 
@@ -605,12 +628,15 @@ static void launch_conv(bool vec4, int grid, cudaStream_t st, const void* u, int
                         const int32_t* seq_len, const int32_t* seq_slot, const int32_t* slot_mapping, const float* q_norm_w,
                         const float* k_norm_w, void* q_out, void* k_cache, void* v_cache, int n_tokens, int n_seqs, int H, int G, int d,
                         int dv, int taps, float eps, int C, const ConvHeadOps& ops) {
-#define CONV4_GO_R(TP, NCH, ROT) conv_headnorm_kvwrite_vec4_kernel<T, TP, NCH, ROT><<<grid, CONV_WARPS * 32, 0, st>>>(static_cast<const T*>(u), u_stride, conv_w, \
+#define CONV4_GO_T(TP, NCH, ROT, TOK) conv_headnorm_kvwrite_vec4_kernel<T, TP, NCH, ROT, TOK><<<grid, CONV_WARPS * 32, 0, st>>>(static_cast<const T*>(u), u_stride, conv_w, \
       static_cast<const T*>(state), tok_seq, positions, seq_start, seq_pos0, seq_slot, slot_mapping, q_norm_w, k_norm_w, \
       static_cast<T*>(q_out), static_cast<T*>(k_cache), static_cast<T*>(v_cache), n_tokens, H, G, d, dv, eps, ops)
+#define CONV4_GO_R(TP, NCH, ROT) do { if (tok == 1) CONV4_GO_T(TP, NCH, ROT, 1); else CONV4_GO_T(TP, NCH, ROT, CONV4_TOKENS); } while (0)
 #define CONV4_GO_N(TP, NCH) do { if (ops.rot_dims > 0) CONV4_GO_R(TP, NCH, true); else CONV4_GO_R(TP, NCH, false); } while (0)
 #define CONV4_GO(TP) do { if (d <= 128 && dv <= 128) CONV4_GO_N(TP, 1); else CONV4_GO_N(TP, 2); } while (0)
-  if (vec4) grid = ((n_tokens + CONV4_TOKENS - 1) / CONV4_TOKENS * (H + 2 * G) + CONV_WARPS - 1) / CONV_WARPS;
+  // rows per warp: one while that leaves the machine short of warps
+  const int tok = static_cast<int64_t>(n_tokens) * (H + 2 * G) <= static_cast<int64_t>(sm_count()) * 64 ? 1 : CONV4_TOKENS;
+  if (vec4) grid = ((n_tokens + tok - 1) / tok * (H + 2 * G) + CONV_WARPS - 1) / CONV_WARPS;
   if (vec4 && taps == 4) CONV4_GO(4);
   else if (vec4 && taps == 3) CONV4_GO(3);
   else if (vec4 && taps == 2) CONV4_GO(2);
@@ -622,6 +648,7 @@ static void launch_conv(bool vec4, int grid, cudaStream_t st, const void* u, int
 #undef CONV4_GO
 #undef CONV4_GO_N
 #undef CONV4_GO_R
+#undef CONV4_GO_T
   if (taps > 1)
     conv_state_update_kernel<T><<<dim3((C + 127) / 128, n_seqs), 128, 0, st>>>(static_cast<const T*>(u), u_stride, static_cast<T*>(state),
         seq_start, seq_pos0, seq_len, seq_slot, n_seqs, C, taps);
