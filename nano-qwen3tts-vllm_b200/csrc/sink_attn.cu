@@ -787,6 +787,7 @@ extern "C" int b2tts_sink_attn(const void* q, const void* k_cache, const void* v
                                             keep_first, softcap, scale, out_f32);
     if (split) B2_CHECK_LAUNCH("sink_attn (one-token rows)");
   }
+  if (use_mma && split) return B2TTS_OK;             // every sequence has its kernel (padding rows come with one-token steps only)
   const int skip = (use_mma ? 1 : 0) | (split ? 2 : 0);
   if (dtype == B2TTS_DTYPE_BF16)
     launch_sink_plain_rep<__nv_bfloat16>(heads / kv_heads, st, q, k_cache, v_cache, out, tok_seq, positions, seq_len, block_tables,
