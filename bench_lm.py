@@ -765,7 +765,7 @@ def zekivik_config(s: dict, moe: bool = False):
     from nano_qwen3tts_vllm_b200.config import ZekivikConfig
     d, H, G = s["dim"], s["heads"], s["kv_heads"]
     mlp = {"kind": "dense", "ff": s["inter"]}
-    rot = {"dims": d, "base": 1e6}
+    rot = {"dims": d, "base": 1e4}
     att = {"type": "attention", "mlp": mlp,
            "mixer": {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "conv": TAPS, "scale": d ** -0.5, "rot": rot}}
     ret = {"type": "retention", "mlp": mlp,
@@ -832,7 +832,7 @@ def bench_zekivik_kernels(device: str) -> dict:
     pps = (DECODE_CTX + PAGE) // PAGE + 1
     dlay, play = layout(DECODE_SEQS, DECODE_CTX, 1, pps), layout(PREFILL_SEQS, 0, PREFILL_LEN, PREFILL_LEN // PAGE)
     n = PREFILL_SEQS * PREFILL_LEN
-    rot = HalfRotaryTable(d, 1e6).to(dev)
+    rot = HalfRotaryTable(d, 1e4).to(dev)
     tables = {id(l): nat.rotary_table(l.positions, rot.freq) for l in (dlay, play)}
     res["rotary_table 8192 tokens"] = entry(timed(lambda: nat.rotary_table(play.positions, rot.freq)), bytes_=n * d * 4)
     # ---- attention: causal, ordinary softmax, a gate per head

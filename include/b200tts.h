@@ -581,7 +581,7 @@ B2TTS_API int b2tts_short_conv_act(const void* u, int64_t ldu, int c_off, const 
                                    const int32_t* tok_seq, const int32_t* positions, const int32_t* seq_start,
                                    const int32_t* seq_pos0, const int32_t* seq_len, const int32_t* seq_slot, void* out, int64_t ldo,
                                    int n_tokens, int n_seqs, int max_new, int channels, int taps, int act, int dtype, void* stream);
-/* Row y [cols] (float) in `groups` equal parts, each divided by its root mean square, times w[c mod w_len]; the gate
+/* Row y [cols] (float) in `groups` equal parts, each divided by its root mean square, times w[c mod w_len] (w null: one); the gate
  * (sigmoid for gate_act 0, SiLU for 1, of gate[r * ldg + c]; null: none) multiplies y before the norm (gate_first) or after. */
 B2TTS_API int b2tts_gated_group_norm(const float* y, const void* gate, int64_t ldg, const float* w, int w_len, int groups,
                                      int gate_act, int gate_first, float eps, void* out, int rows, int cols, int dtype, void* stream);
