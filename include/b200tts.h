@@ -264,9 +264,18 @@ B2TTS_API int b2tts_frame_advance(const int64_t* code0, int eos_id, int32_t* act
 #define B2TTS_GEMM_SILU_MUL 2
 #define B2TTS_GEMM_RELU_SQ  3
 #define B2TTS_GEMM_GELU_MUL 4
+#define B2TTS_GEMM_CLAMPED_GATE 5
 #define B2TTS_PACK_PLAIN    0
 #define B2TTS_PACK_GATE_UP  1
 B2TTS_API int    b2tts_gemm_bf16_supported(int m, int n, int k);
+/* The bias epilogue with a float output (the sums leave unrounded; out_row_stride in floats), and
+ * out[m, n/2] = bf16(g * sigmoid(alpha g) * (u + 1)), g = min(gate, limit), u = clamp(up, -limit, limit) over a
+ * B2TTS_PACK_GATE_UP weight (epilogue B2TTS_GEMM_CLAMPED_GATE, which only this entry point takes). */
+B2TTS_API int    b2tts_gemm_f32out_bf16(const void* x, int64_t x_row_stride, const void* w_packed, const void* bias, float* out,
+                                        int64_t out_row_stride, int m, int n, int k, int splits, int pdl, void* stream);
+B2TTS_API int    b2tts_gemm_clamped_gate_bf16(const void* x, int64_t x_row_stride, const void* w_packed, void* out,
+                                              int64_t out_row_stride, int m, int n, int k, float limit, float alpha,
+                                              int splits, int pdl, void* stream);
 B2TTS_API size_t b2tts_gemm_packed_bytes(int n, int k);
 B2TTS_API int    b2tts_gemm_pack_weight(const void* weight, int64_t weight_row_stride, void* packed,
                                         int n, int k, int mode, void* stream);
@@ -468,17 +477,23 @@ B2TTS_API int b2tts_window_sigmoid_attn(const void* q, const void* k_cache, cons
 /* Top-k router, in float.  mode 0: scores = sigmoid(h router^T), top_w = score / (sum of the chosen + 1e-20) * scale.
  * mode 1: scores = h router^T + bias (bias may be null), top_w = softmax over the chosen scores only, * scale.
  * mode 2: scores = softmax(h router^T) over all experts, the choice is made on score + bias, top_w = the chosen scores
- * * scale (not renormalised).  top_idx [n, top] the `top` largest (ties: lower index); then the (token, choice) pairs grouped by expert:
+ * * scale (not renormalised).  groups > 1: equal groups of neighbouring experts, scored by their largest choice score; only experts
+ * of the groups_keep best groups can be chosen (top <= groups_keep * experts / groups).  top_idx [n, top] the `top` largest (ties: lower index); then the (token, choice) pairs grouped by expert:
  * offsets [experts + 1], sorted_pair [n * top] (pair = token * top + choice; order inside a group unspecified). */
 B2TTS_API int b2tts_moe_route(const void* h, const float* router, int32_t* top_idx, float* top_w, int32_t* offsets,
                               int32_t* sorted_pair, int n_tokens, int cols, int experts, int top, float scale,
-                              const float* bias, int mode, int dtype, void* stream);
+                              const float* bias, int mode, int groups, int groups_keep, int dtype, void* stream);
 /* C[out_row(s), :] = act(A[in_row(s), :] W[e]^T) for s in offsets[e] .. offsets[e+1], W [experts, n, k];
  * in_row(s) = sorted_pair[s] / top if in_by_token else s; out_row(s) = sorted_pair[s] if out_by_pair else s;
  * act 0 = none, 1 = squared ReLU; float accumulation. */
 B2TTS_API int b2tts_grouped_gemm(const void* a, int64_t lda, const void* w, void* c, int64_t ldc, const int32_t* offsets,
                                  const int32_t* sorted_pair, int n_pairs, int experts, int n, int k, int top, int in_by_token,
                                  int out_by_pair, int act, int dtype, void* stream);
+/* Gated experts: w [experts, 2 ff, k] = [gate; up] per expert, c[s, ff] = g * sigmoid(alpha g) * (u + 1) with g = min(gate, limit),
+ * u = clamp(up, -limit, limit) of row s of the sorted pairs (input row: its token).  bf16; ff and k multiples of 8. */
+B2TTS_API int b2tts_grouped_gemm_gated(const void* a, int64_t lda, const void* w, void* c, int64_t ldc, const int32_t* offsets,
+                                       const int32_t* sorted_pair, int n_pairs, int experts, int ff, int k, int top, float limit,
+                                       float alpha, void* stream);
 
 /* ---- decoders with latent attention, token shift and a norm on each sublayer's output (csrc/latent_ops.cu, latent_attn.cu).
  * `dtype` is the activation / cache type (B2TTS_DTYPE_*); x is the float residual stream [rows, cols]. */
@@ -515,9 +530,10 @@ B2TTS_API int b2tts_latent_attn_splits(int n_seqs, int max_new, int heads);
 B2TTS_API size_t b2tts_latent_attn_workspace_floats(int n_seqs, int max_new, int heads, int kv_rank, int splits);
 /* How many bounded waits for a key tile ran out inside the tensor-core kernel since load (0 in a healthy run); synchronises. */
 B2TTS_API int b2tts_latent_attn_timeouts(void);
-/* out[t, h * vdim + d] = v[t * v_tok + h * v_head + d] * sigmoid(gate[t * ldg + h * vdim + d]) (gate null: the copy alone). */
+/* out[t, h * vdim + d] = v[t * v_tok + h * v_head + d] * sigmoid(gate[t * ldg + h * vdim + d]), per_head != 0: * sigmoid(gate[t * ldg + h])
+ * (gate null: the copy alone). */
 B2TTS_API int b2tts_gate_heads(const void* v, int64_t v_tok, int64_t v_head, const void* gate, int64_t ldg, void* out, int n,
-                               int heads, int vdim, int dtype, void* stream);
+                               int heads, int vdim, int per_head, int dtype, void* stream);
 /* y = a + sum_k zw[:, k] z[:, k] (a or z may be null); x += w * y / sqrt(mean over the group (y^2) + eps), the row cut into
  * `groups` equal consecutive parts; copy (optional) = the new x in the activation type. */
 B2TTS_API int b2tts_group_norm_residual(float* x, const void* a, const void* z, const float* zw, int top, const float* w, int groups,
@@ -559,18 +575,27 @@ B2TTS_API int b2tts_attn_prep(const void* u, int64_t ldu, int q_off, int k_off, 
                               const int32_t* positions, const int32_t* slot_mapping, void* q_out, void* k_cache, void* v_cache,
                               int n_tokens, int heads, int kv_heads, int dim, int vdim, float eps, int interleaved, int v_heads,
                               int dtype, void* stream);
+/* The same preparation for heads that are normed one by one: q and k heads (with their biases) are divided by the root mean square
+ * of the HEAD and multiplied by q_norm_w / k_norm_w [dim] (both null: no norm), THEN the first rot_dims coordinates are turned by
+ * the angles of `rot` [n, rot_dims] (b2tts_rotary_table: cosines, then sines; interleaved != 0: coordinate 2i with 2i + 1, else i
+ * with i + rot_dims/2).  q -> q_out[t]; k and v (with its bias) -> the caches at slot_mapping[t] (< 0: padding). */
+B2TTS_API int b2tts_attn_head_prep(const void* u, int64_t ldu, int q_off, int k_off, int v_off, const float* q_bias, const float* k_bias,
+                                   const float* v_bias, const float* q_norm_w, const float* k_norm_w, const float* rot, int rot_dims,
+                                   int interleaved, const int32_t* slot_mapping, void* q_out, void* k_cache, void* v_cache,
+                                   int n_tokens, int heads, int kv_heads, int dim, int vdim, float eps, int dtype, void* stream);
 /* Softmax attention with exp(sink[h]) added to the denominator (sink null: none) over the paged cache, this step's keys
  * included.  Token i sees key j <= i with j >= max(0, i - mask + 1) (mask_kind 0, a sliding window) or j >= floor(i / mask) *
  * mask (mask_kind 1, chunks counted from position 0); mask <= 0: every j <= i.  keep_first F > 0: keys j < F stay visible
  * behind the mask.  softcap c > 0: a scaled score s becomes c tanh(s / c).  v_heads: value heads in v_cache, key head g reads
  * value head g mod v_heads (v_heads == kv_heads: one each).  out_f32 != 0 with bf16 inputs: out is a float tensor (results not
  * rounded to 16 bits).  gate (optional): element (t, h) at
- * gate[t * ldg + h]; the head's output is multiplied by its sigmoid.  q [n, heads*dim], out [n, heads*vdim].  max_new >= every
+ * gate[t * ldg + h]; the head's output is multiplied by its sigmoid (gate_el != 0: output element (t, h, c) by that of
+ * gate[t * ldg + h * vdim + c]).  q [n, heads*dim], out [n, heads*vdim].  max_new >= every
  * seq_len[b].  path 0 = choose (bf16 prompt portions with head sizes the tensor-core kernel is built for run there, everything
  * else in the plain kernel), 1 = the plain kernel, 2 = the tensor-core kernel for prompt portions (fails if the sizes do not fit). */
 B2TTS_API int b2tts_sink_attn(const void* q, const void* k_cache, const void* v_cache, void* out, const int32_t* tok_seq,
                               const int32_t* positions, const int32_t* seq_start, const int32_t* seq_pos0, const int32_t* seq_len,
-                              const int32_t* block_tables, int64_t bt_stride, const float* sink, const void* gate, int64_t ldg,
+                              const int32_t* block_tables, int64_t bt_stride, const float* sink, const void* gate, int64_t ldg, int gate_el,
                               int n_tokens, int n_seqs, int max_new, int heads, int kv_heads, int v_heads, int dim, int vdim,
                               int page, int mask_kind, int mask, int keep_first, float softcap, float scale, int dtype, int path,
                               int out_f32, void* stream);
@@ -637,6 +662,20 @@ B2TTS_API int b2tts_diff_combine(const void* maps, void* out, float lambda, floa
                                  int maps_f32, int dtype, void* stream);
 /* In place: y <- cap * tanh(y / cap). */
 B2TTS_API int b2tts_tanh_cap(float* y, int64_t n, float cap, void* stream);
+
+/* ---- decoders whose norms are dynamic tanh, D(v) = tanh(alpha[0] v) * w + b (csrc/tanh_ops.cu) ----
+ * x[r] (init != 0: starting from row index[r] of `table`) += mult * D_out(a[r] + sum_k zw[r, k] * z[r * top + k]) (a and z may each be
+ * null; both null: no update).  h[r] = D_in(x[r]) when h != null.  cat != null: the operand of a pass's input projection, bf16
+ * [rows, 3 cols] = x as two bf16 numbers hi | lo, then the table row, or float [rows, 2 cols] = x | the table row. */
+B2TTS_API int b2tts_tanh_residual(float* x, const void* table, const int32_t* index, int table_rows, const void* a, const void* z,
+                                  const float* zw, int top, const float* out_w, const float* out_b, const float* out_alpha, float mult,
+                                  const float* in_w, const float* in_b, const float* in_alpha, void* h, void* cat, int rows, int cols,
+                                  int init, int dtype, void* stream);
+/* out[i] = D(x[rows_idx[i]]) (rows_idx null: row i). */
+B2TTS_API int b2tts_tanh_gather(const float* x, const int32_t* rows_idx, void* out, const float* w, const float* b, const float* alpha,
+                                int rows, int cols, int dtype, void* stream);
+/* gu [rows, 2 ff] = [gate | up]: y[rows, ff] = g * sigmoid(alpha g) * (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit). */
+B2TTS_API int b2tts_clamped_gate_mul(const void* gu, void* y, int64_t rows, int ff, float limit, float alpha, int dtype, void* stream);
 
 /* ---- decoders with gated residuals and fixed-decay retention (csrc/gated_ops.cu, csrc/retention.cu) ----
  * x[r] (init != 0: starting from zero) += sigmoid(z[r * ldz + c] + zb[c]) * y[r] (z null: y as it is; y null: nothing), then += row

@@ -65,6 +65,8 @@ def _load():
         "b2tts_gemm_packed_bytes": (Z, [I, I]),
         "b2tts_gemm_pack_weight": (I, [P, L, P, I, I, I, P]),
         "b2tts_gemm_bf16": (I, [P, L, P, P, P, L, P, L, I, I, I, I, I, I, I, P]),
+        "b2tts_gemm_f32out_bf16": (I, [P, L, P, P, P, L, I, I, I, I, I, P]),
+        "b2tts_gemm_clamped_gate_bf16": (I, [P, L, P, P, L, I, I, I, F, F, I, I, P]),
         "b2tts_gemm_ssq_slots": (I, [I, I, I, I]),
         "b2tts_fused_decode_attn_workspace_bytes": (Z, [I, I, I, I]),
         "b2tts_fused_decode_attn": (I, [P, L, P, L, P, L, P, P, F, P, L, P, P, F, P, P, P, P, I, P, P, P, Z,
@@ -91,7 +93,12 @@ def _load():
         "b2tts_retention": (I, [P, L, P, L, P, L, P, I, P, F, P, P, L, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, P]),
         "b2tts_retention_scratch": (I, [I, I, I, I, I, I, I]),
         "b2tts_window_sigmoid_attn": (I, [P, P, P, P, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, I, P]),
-        "b2tts_moe_route": (I, [P, P, P, P, P, P, I, I, I, I, F, P, I, I, P]),
+        "b2tts_moe_route": (I, [P, P, P, P, P, P, I, I, I, I, F, P, I, I, I, I, P]),
+        "b2tts_grouped_gemm_gated": (I, [P, L, P, P, L, P, P, I, I, I, I, I, F, F, P]),
+        "b2tts_tanh_residual": (I, [P, P, P, I, P, P, P, I, P, P, P, F, P, P, P, P, P, I, I, I, I, P]),
+        "b2tts_tanh_gather": (I, [P, P, P, P, P, P, I, I, I, P]),
+        "b2tts_clamped_gate_mul": (I, [P, P, L, I, F, F, I, P]),
+        "b2tts_attn_head_prep": (I, [P, L, I, I, I, P, P, P, P, P, P, I, I, P, P, P, P, I, I, I, I, I, F, I, P]),
         "b2tts_embed_scale": (I, [P, P, P, I, I, I, F, I, P]),
         "b2tts_token_shift": (I, [P, P, P, P, P, P, P, P, P, I, I, I, P]),
         "b2tts_latent_prep": (I, [P, L, I, I, P, P, P, P, F, P, P, P, I, I, I, I, I, F, I, P]),
@@ -99,7 +106,7 @@ def _load():
         "b2tts_latent_attn_splits": (I, [I, I, I]),
         "b2tts_latent_attn_timeouts": (I, []),
         "b2tts_latent_attn_workspace_floats": (Z, [I, I, I, I, I]),
-        "b2tts_gate_heads": (I, [P, L, L, P, L, P, I, I, I, I, P]),
+        "b2tts_gate_heads": (I, [P, L, L, P, L, P, I, I, I, I, I, P]),
         "b2tts_group_norm_residual": (I, [P, P, P, P, I, P, I, F, P, I, I, I, P]),
         "b2tts_gather_group_norm": (I, [P, P, P, P, I, F, I, I, I, P]),
         "b2tts_xielu": (I, [P, P, P, L, I, I, P]),
@@ -108,7 +115,7 @@ def _load():
         "b2tts_stream_mix_norm": (I, [P, P, P, F, F, P, P, P, P, P, I, I, I, F, I, P]),
         "b2tts_stream_gather_norm": (I, [P, P, P, P, P, I, I, I, F, I, P]),
         "b2tts_attn_prep": (I, [P, L, I, I, I, P, P, P, P, P, P, I, P, P, P, P, P, I, I, I, I, I, F, I, I, I, P]),
-        "b2tts_sink_attn": (I, [P, P, P, P, P, P, P, P, P, P, L, P, P, L, I, I, I, I, I, I, I, I, I, I, I, I, F, F, I, I, I, P]),
+        "b2tts_sink_attn": (I, [P, P, P, P, P, P, P, P, P, P, L, P, P, L, I, I, I, I, I, I, I, I, I, I, I, I, I, F, F, I, I, I, P]),
         "b2tts_gated_linear_scan": (I, [P, L, P, L, P, L, P, L, P, F, P, P, P, P, P, P, P, I, I, I, I, I, I, P]),
         "b2tts_sandwich_residual": (I, [P, P, P, I, P, P, P, F, P, P, P, I, I, P, P, P, P, I, I, I, F, I, P]),
         "b2tts_polynorm": (I, [P, P, I, I, F, I, P]),
@@ -545,6 +552,31 @@ def gemm_bf16(x, packed, n, bias=None, residual=None, epilogue=GEMM_BIAS, roundi
     return out
 
 
+def gemm_f32out(x, packed, n, bias=None, out=None, splits=0, pdl=False):
+    """float [M, n] = x[M, K] @ W[n, K]^T (+ bias): the float sums leave unrounded."""
+    _cuda(x, BF16, "x")
+    m, k = x.shape
+    assert x.stride(1) == 1
+    if out is None:
+        out = torch.empty(m, n, dtype=F32, device=x.device)
+    _cuda(out, F32, "out")
+    _check(_load().b2tts_gemm_f32out_bf16(x.data_ptr(), x.stride(0), packed.data_ptr(), _ptr(bias), out.data_ptr(), out.stride(0), m, n, k,
+                                          int(splits), int(bool(pdl)), _stream()), "gemm_f32out_bf16")
+    return out
+
+
+def gemm_clamped_gate(x, packed, n, limit, alpha, splits=0, pdl=False):
+    """[M, n / 2] = the clamped gated product over a [gate; up] weight packed with PACK_GATE_UP, in the GEMM's epilogue."""
+    _cuda(x, BF16, "x")
+    m, k = x.shape
+    if x.stride(1) != 1:
+        x = x.contiguous()
+    out = torch.empty(m, n // 2, dtype=BF16, device=x.device)
+    _check(_load().b2tts_gemm_clamped_gate_bf16(x.data_ptr(), x.stride(0), packed.data_ptr(), out.data_ptr(), out.stride(0), m, n, k,
+                                                float(limit), float(alpha), int(splits), int(bool(pdl)), _stream()), "gemm_clamped_gate_bf16")
+    return out
+
+
 # ------------------------------------------------------------------------------------------ a7 x 4: GEMM chain
 class GemmOp(ctypes.Structure):
     """``b2tts_gemm_op`` (include/b200tts.h)."""
@@ -806,10 +838,12 @@ def window_sigmoid_attn(q, k_cache, v_cache, out, lay, r1, r2, pb, heads, kv_hea
 ROUTE_SIGMOID, ROUTE_SOFTMAX_CHOSEN, ROUTE_SOFTMAX_ALL = 0, 1, 2
 
 
-def moe_route(h, router, top_idx, top_w, offsets, sorted_pair, top, scale, bias=None, softmax_chosen=False, mode=None):
+def moe_route(h, router, top_idx, top_w, offsets, sorted_pair, top, scale, bias=None, softmax_chosen=False, mode=None, groups=1,
+              groups_keep=1):
     """``mode`` ROUTE_SIGMOID: sigmoid scores divided by the sum of the chosen; ROUTE_SOFTMAX_CHOSEN (= ``softmax_chosen``):
     scores are the logits (+ ``bias``) and the weights their softmax over the chosen ones; ROUTE_SOFTMAX_ALL: scores are
-    the softmax over all logits, ``bias`` enters the choice only and the weights are the chosen scores as they are."""
+    the softmax over all logits, ``bias`` enters the choice only and the weights are the chosen scores as they are.
+    ``groups`` > 1: only experts of the ``groups_keep`` groups of neighbours with the largest choice scores can be chosen."""
     if mode is None:
         mode = ROUTE_SOFTMAX_CHOSEN if softmax_chosen else ROUTE_SIGMOID
     dt = _act(h, "h")
@@ -819,7 +853,7 @@ def moe_route(h, router, top_idx, top_w, offsets, sorted_pair, top, scale, bias=
     n, cols = h.shape
     _check(_load().b2tts_moe_route(h.data_ptr(), router.data_ptr(), top_idx.data_ptr(), top_w.data_ptr(), offsets.data_ptr(),
                                    sorted_pair.data_ptr(), n, cols, router.shape[0], top, scale, _ptr(bias), int(mode),
-                                   dt, _stream()), "moe_route")
+                                   groups, groups_keep, dt, _stream()), "moe_route")
 
 
 def grouped_gemm(a, w, c, offsets, sorted_pair, n_pairs, top, in_by_token, out_by_pair, act):
@@ -830,6 +864,35 @@ def grouped_gemm(a, w, c, offsets, sorted_pair, n_pairs, top, in_by_token, out_b
     _check(_load().b2tts_grouped_gemm(a.data_ptr(), a.stride(0), w.data_ptr(), c.data_ptr(), c.stride(0), offsets.data_ptr(),
                                       sorted_pair.data_ptr(), n_pairs, e, n, k, top, int(in_by_token), int(out_by_pair), int(act),
                                       dt, _stream()), "grouped_gemm")
+
+
+GATE_SIGMOID_SCALE = 1.702      # of the clamped gated product
+
+
+def clamped_gate_mul(gu, limit, alpha=GATE_SIGMOID_SCALE, out=None):
+    """gu [rows, 2 ff] = [gate | up] -> g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)."""
+    dt = _act(gu, "gu")
+    ff = gu.shape[1] // 2
+    if out is None:
+        out = torch.empty(gu.shape[0], ff, dtype=gu.dtype, device=gu.device)
+    _check(_load().b2tts_clamped_gate_mul(gu.data_ptr(), out.data_ptr(), gu.shape[0], ff, limit, alpha, dt, _stream()), "clamped_gate_mul")
+    return out
+
+
+def grouped_gemm_gated(a, w, c, offsets, sorted_pair, n_pairs, top, limit, alpha=GATE_SIGMOID_SCALE):
+    """c [n_pairs, ff] <- the clamped gated product of every sorted pair's expert: w [E, 2 ff, K] = [gate; up] per expert.  bf16
+    with ff and K multiples of 8 runs as one launch; anything else is the grouped product followed by the activation kernel."""
+    _act(a, "a")
+    e, n, k = w.shape
+    ff = n // 2
+    if a.dtype == BF16 and ff % 8 == 0 and k % 8 == 0:
+        assert w.dtype == BF16 and c.dtype == BF16 and w.is_contiguous() and c.is_contiguous()
+        _check(_load().b2tts_grouped_gemm_gated(a.data_ptr(), a.stride(0), w.data_ptr(), c.data_ptr(), c.stride(0), offsets.data_ptr(),
+                                                sorted_pair.data_ptr(), n_pairs, e, ff, k, top, limit, alpha, _stream()), "grouped_gemm_gated")
+        return c
+    gu = torch.empty(n_pairs, n, dtype=a.dtype, device=a.device)
+    grouped_gemm(a, w, gu, offsets, sorted_pair, n_pairs, top, in_by_token=True, out_by_pair=False, act=0)
+    return clamped_gate_mul(gu, limit, alpha, out=c)
 
 
 # ------------------------------------------------------------------------------------------ latent-attention decoders
@@ -886,12 +949,13 @@ def latent_attn_timeouts() -> int:
     return _load().b2tts_latent_attn_timeouts()
 
 
-def gate_heads(v, v_strides, gate, out, heads, vdim):
-    """out [n, heads * vdim] <- v (token / head strides given) * sigmoid(gate) (``gate``: a column slice, or None)."""
+def gate_heads(v, v_strides, gate, out, heads, vdim, per_head=False):
+    """out [n, heads * vdim] <- v (token / head strides given) * sigmoid(gate) (``gate``: a column slice, or None; ``per_head``:
+    one column per head)."""
     dt = _act(out, "out")
     assert v.dtype == out.dtype and (gate is None or (gate.dtype == out.dtype and gate.stride(1) == 1))
     _check(_load().b2tts_gate_heads(v.data_ptr(), v_strides[0], v_strides[1], _ptr(gate), 0 if gate is None else gate.stride(0),
-                                    out.data_ptr(), out.shape[0], heads, vdim, dt, _stream()), "gate_heads")
+                                    out.data_ptr(), out.shape[0], heads, vdim, int(per_head), dt, _stream()), "gate_heads")
 
 
 def group_norm_residual(x, a, z, zw, w, groups, eps, copy, dtype):
@@ -988,6 +1052,21 @@ def attn_prep(u, q_off, k_off, v_off, q_bias, k_bias, v_bias, q_norm_w, k_norm_w
                                    kv_heads if v_heads is None else v_heads, dt, _stream()), "attn_prep")
 
 
+def attn_head_prep(u, q_off, k_off, v_off, q_bias, k_bias, v_bias, q_norm_w, k_norm_w, rot, interleaved, lay, q_out, k_cache, v_cache,
+                   heads, kv_heads, dim, vdim, eps):
+    """Biases, RMS norm of every q and k head (weights [dim], or None), then rotation by the step's ``rotary_table`` ``rot`` (None: no
+    rotation); k and v go to their cache slots."""
+    dt = _act(q_out, "q_out")
+    assert u.dtype == q_out.dtype and u.stride(1) == 1 and k_cache.dtype == u.dtype and v_cache.dtype == u.dtype
+    for t in (q_bias, k_bias, v_bias, q_norm_w, k_norm_w):
+        assert t is None or (t.dtype == F32 and t.is_contiguous())
+    assert rot is None or (rot.dtype == F32 and rot.is_contiguous() and rot.shape[0] >= lay.n_tokens)
+    _check(_load().b2tts_attn_head_prep(u.data_ptr(), u.stride(0), q_off, k_off, v_off, _ptr(q_bias), _ptr(k_bias), _ptr(v_bias),
+                                        _ptr(q_norm_w), _ptr(k_norm_w), _ptr(rot), 0 if rot is None else rot.shape[1], int(interleaved),
+                                        lay.slot_mapping.data_ptr(), q_out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
+                                        lay.n_tokens, heads, kv_heads, dim, vdim, eps, dt, _stream()), "attn_head_prep")
+
+
 MASK_WINDOW, MASK_CHUNK = 0, 1
 
 
@@ -995,8 +1074,8 @@ SINK_ATTN_AUTO, SINK_ATTN_PLAIN, SINK_ATTN_TENSOR = 0, 1, 2
 
 
 def sink_attn(q, k_cache, v_cache, out, lay, sink, gate, heads, kv_heads, dim, vdim, page, mask_kind, mask, scale, path=SINK_ATTN_AUTO,
-              v_heads=None, keep_first=0, softcap=0.0):
-    """``gate``: a column slice [n, heads] of the merged projection (or None).  ``sink`` None: an ordinary softmax.
+              v_heads=None, keep_first=0, softcap=0.0, gate_el=False):
+    """``gate``: a column slice [n, heads], or [n, heads * vdim] with ``gate_el``, of the merged projection (or None).  ``sink`` None: an ordinary softmax.
     ``v_heads``: value heads in the cache (key head g reads value head g mod v_heads; default ``kv_heads``);
     ``keep_first``: keys below this position stay visible behind the mask; ``softcap`` c > 0: scores become c tanh(s / c).
     ``out`` may be a float tensor beside bfloat16 inputs: the results are then not rounded to 16 bits."""
@@ -1006,7 +1085,7 @@ def sink_attn(q, k_cache, v_cache, out, lay, sink, gate, heads, kv_heads, dim, v
     _check(_load().b2tts_sink_attn(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), lay.tok_seq.data_ptr(),
                                    lay.positions.data_ptr(), lay.seq_start.data_ptr(), lay.seq_pos0.data_ptr(), lay.seq_len.data_ptr(),
                                    lay.block_tables.data_ptr(), lay.block_tables.stride(0), _ptr(sink), _ptr(gate),
-                                   0 if gate is None else gate.stride(0), lay.n_tokens, lay.n_seqs, lay.max_new, heads, kv_heads,
+                                   0 if gate is None else gate.stride(0), int(gate_el), lay.n_tokens, lay.n_seqs, lay.max_new, heads, kv_heads,
                                    kv_heads if v_heads is None else v_heads, dim, vdim, page, mask_kind, mask, keep_first, softcap,
                                    scale, dt, path, int(out.dtype == F32 and q.dtype != F32), _stream()), "sink_attn")
 
@@ -1167,6 +1246,42 @@ def gated_residual(x, *, y=None, z=None, zb=None, table=None, index=None, add=No
                                         0 if table is None else table.shape[0], _ptr(add), _ptr(w), _ptr(h), n, cols, int(init), eps,
                                         DTYPE_CODE[dtype], _stream()), "gated_residual")
     return h
+
+
+# ------------------------------------------------------------------------------------------ dynamic tanh norms
+def tanh_residual(x, *, table=None, index=None, init=False, a=None, z=None, zw=None, post=None, mult=1.0, pre=None, want_cat=False, dtype=None):
+    """x (float [n, cols], in place; ``init``: starting from ``table[index]``) += mult * D_post(a + sum_k zw[:, k] z[:, k]) when a sublayer's
+    result is given.  ``post`` / ``pre``: (w, b, alpha) float tensors of a dynamic tanh.  Returns D_pre(x) in the activation type when
+    ``pre`` is given; with ``want_cat`` the operand of a pass's input projection: bf16 [n, 3 cols] = x as hi | lo, then the table row,
+    or float [n, 2 cols] = x | the table row."""
+    _cuda(x, F32, "x")
+    n, cols = x.shape
+    dtype = dtype or next(t.dtype for t in (a, z, table) if t is not None)
+    assert x.is_contiguous() and not (pre is not None and want_cat)
+    for t in (table, a, z):
+        assert t is None or (t.dtype == dtype and t.is_contiguous() and t.shape[-1] == cols)
+    for norm in (post, pre):
+        assert norm is None or (all(t.dtype == F32 and t.is_contiguous() for t in norm) and norm[0].numel() == norm[1].numel() == cols)
+    ow, ob, oa = post if post is not None else (None, None, None)
+    iw, ib, ia = pre if pre is not None else (None, None, None)
+    h = torch.empty(n, cols, dtype=dtype, device=x.device) if pre is not None else None
+    cat = torch.empty(n, (3 if dtype == BF16 else 2) * cols, dtype=dtype, device=x.device) if want_cat else None
+    _check(_load().b2tts_tanh_residual(x.data_ptr(), _ptr(table), _ptr(index), 0 if table is None else table.shape[0], _ptr(a), _ptr(z),
+                                       _ptr(zw), 0 if z is None else zw.shape[1], _ptr(ow), _ptr(ob), _ptr(oa), mult, _ptr(iw), _ptr(ib),
+                                       _ptr(ia), _ptr(h), _ptr(cat), n, cols, int(init), DTYPE_CODE[dtype], _stream()), "tanh_residual")
+    return cat if want_cat else h
+
+
+def tanh_gather(x, rows, norm, dtype, out=None):
+    """out[i] = D(x[rows[i]]) (``rows`` None: every row); ``norm`` = (w, b, alpha)."""
+    _cuda(x, F32, "x")
+    n = x.shape[0] if rows is None else rows.shape[0]
+    if out is None:
+        out = torch.empty(n, x.shape[1], dtype=dtype, device=x.device)
+    w, b, alpha = norm
+    _check(_load().b2tts_tanh_gather(x.data_ptr(), _ptr(rows), out.data_ptr(), w.data_ptr(), b.data_ptr(), alpha.data_ptr(), n, x.shape[1],
+                                     DTYPE_CODE[dtype], _stream()), "tanh_gather")
+    return out
 
 
 def gelu_mul(gu, out=None):

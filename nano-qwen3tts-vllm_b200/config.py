@@ -122,11 +122,16 @@ class FeedForwardSpec:
     top: int = 0
     router_scale: float = 1.0
     act: str = "relu2"             # "relu2": relu(up)^2;  "xielu": two learned numbers;  "silu_gate": silu(gate) * up;
-                                   # "polynorm": a N(z) + b N(z^2) + c N(z^3) + e with four learned numbers
+                                   # "polynorm": a N(z) + b N(z^2) + c N(z^3) + e with four learned numbers;
+                                   # "clamped_gate": g sigmoid(1.702 g) (u + 1), g = min(gate, limit), u = clamp(up, +-limit)
     bias: bool = False             # dense projections carry biases
     router: str = "sigmoid"        # "sigmoid": scores / their sum;  "softmax_chosen": logits + bias, softmax over the chosen;
                                    # "softmax_all": softmax over all outputs, a correction enters the choice only
     identity: int = 0              # router outputs beyond ``experts`` that stand for experts returning their input
+    limit: float = 0.0             # the clamp of "clamped_gate"
+    groups: int = 1                # experts form this many equal groups of neighbours, ...
+    groups_keep: int = 1           # ... and only those of the groups with the largest scores can be chosen
+    shared: object | None = None   # FeedForwardSpec of an expert that runs for every token beside the chosen ones
 
 
 @dataclass
@@ -225,6 +230,7 @@ class LatentMixerSpec:
     scale: float
     rot: RotarySpec
     gate: bool
+    head_gate: bool = False        # one gate per head instead of one per output element
 
     @property
     def cache_width(self) -> int:
@@ -360,6 +366,8 @@ class SinkAttentionSpec:
     conv: int = 0                  # taps of a short causal convolution on every channel of q, k and v (0: none)
     unit_qk: bool = False          # after rotation every q and k head is divided by its root mean square (no weight)
     unit_v: bool = False           # so is every value head
+    head_norm: bool = False        # RMS norm of every q and k head (one weight of ``dim`` for q, one for k) before the rotation
+    element_gate: bool = False     # one sigmoid gate per output element
 
 
 @dataclass
@@ -697,6 +705,16 @@ class ZekivikLayerSpec:
     raw: dict = field(default_factory=dict, repr=False)      # the layer's entry as read (kept for to_dict)
 
 
+def loop_runs(n: int, loop: dict | None) -> list[tuple[int, int | None]]:
+    """(layer index, number of the pass that starts right before it or None) of every run of ``n`` layers, the range
+    ``loop`` = {"start", "stop", "times"} repeated in a row."""
+    if not loop:
+        return [(i, None) for i in range(n)]
+    a, b = loop["start"], loop["stop"]
+    looped = [(i, t if i == a else None) for t in range(loop["times"]) for i in range(a, b)]
+    return [(i, None) for i in range(a)] + looped + [(i, None) for i in range(b, n)]
+
+
 @dataclass
 class ZekivikConfig:
     """``config.json`` of a Zekivik checkpoint: a decoder-only token model over one 32-bit residual stream whose sublayers
@@ -764,16 +782,112 @@ class ZekivikConfig:
 
     def runs(self) -> list[tuple[int, int | None]]:
         """(layer index, number of the pass that starts right before it or None) of every layer run, in order."""
-        n = len(self.layers)
-        if not self.loop:
-            return [(i, None) for i in range(n)]
-        a, b, times = self.loop["start"], self.loop["stop"], self.loop["times"]
-        looped = [(i, t if i == a else None) for t in range(times) for i in range(a, b)]
-        return [(i, None) for i in range(a)] + looped + [(i, None) for i in range(b, n)]
+        return loop_runs(len(self.layers), self.loop)
 
     def to_dict(self) -> dict:
         out = {"architecture": self.architecture, "vocab": self.vocab, "width": self.width, "norm": {"eps": self.norm_eps},
                "layers": [dict(l.raw) for l in self.layers]}
+        if self.loop:
+            out["loop"] = dict(self.loop)
+        return out
+
+
+@dataclass
+class GekavikLayerSpec:
+    type: str                      # "attention" | "latent_attention"
+    mixer: object                  # SinkAttentionSpec | LatentMixerSpec
+    mlp: FeedForwardSpec | None
+    raw: dict = field(default_factory=dict, repr=False)      # the layer's entry as read (kept for to_dict)
+
+
+@dataclass
+class GekavikConfig:
+    """``config.json`` of a Gekavik checkpoint: a decoder-only token model over one 32-bit residual stream whose sublayers
+    are normed on the way in and on the way out by dynamic tanh.  Layers are listed one by one with their own sizes: biased
+    rotary window attention with head norms, kept first keys and an element-wise output gate, or windowed latent attention
+    without positions and with a gate per head; feed-forwards are mixtures of clamped gated experts with group-limited
+    routing and a shared expert, or absent.  ``loop`` repeats a range of layers with the same weights, each pass over a
+    cache of its own; in front of every pass the stream and the token's embedding go through a projection and get a vector
+    of the pass."""
+    architecture: str
+    vocab: int
+    width: int
+    norm_eps: float
+    residual_mult: float
+    layers: list
+    loop: dict | None              # {"start", "stop", "times"}
+    max_positions = None           # positions enter through rotations only: no table bounds them
+
+    page_multiple = 16
+
+    @staticmethod
+    def _attention(m: dict, i: int) -> SinkAttentionSpec:
+        mask, r = m.get("mask") or {}, m.get("rot")
+        rot = RotarySpec(int(r["dims"]), float(r["base"])) if r and int(r["dims"]) else None
+        spec = SinkAttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                                 mask_kind="window", mask_size=int(mask.get("size") or 0), scale=float(m["scale"]), rot=rot, bias=True,
+                                 keep_first=int(mask.get("keep_first") or 0), sink="none", head_norm=True, element_gate=True)
+        if spec.heads % spec.kv_heads:
+            raise ValueError(f"layer {i}: {spec.heads} heads over {spec.kv_heads} key/value heads")
+        if rot is not None and (rot.dims % 2 or rot.dims > spec.dim):
+            raise ValueError(f"layer {i}: {rot.dims} rotated coordinates in a head of {spec.dim}")
+        return spec
+
+    @staticmethod
+    def _latent(m: dict, i: int) -> LatentMixerSpec:
+        if m.get("rot_dim"):
+            raise ValueError(f"layer {i}: latent attention of this family has no rotated part")
+        mask = m.get("mask") or {}
+        return LatentMixerSpec(heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=0, vdim=int(m["vdim"]), kv_rank=int(m["kv_rank"]),
+                               q_rank=int(m["q_rank"]), window=int(mask.get("size") or 0), scale=float(m["scale"]),
+                               rot=RotarySpec(0, 1.0), gate=True, head_gate=True)
+
+    @staticmethod
+    def _moe(f: dict, i: int) -> FeedForwardSpec:
+        if f["kind"] != "moe":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
+        ro, g, sh = f["router"], f["router"].get("groups") or {}, f.get("shared")
+        shared = FeedForwardSpec("dense", int(sh["ff"]), act="clamped_gate", limit=float(sh["limit"])) if sh else None
+        spec = FeedForwardSpec("moe", int(f["expert"]["ff"]), int(ro["experts"]), int(ro["top"]), act="clamped_gate", router="softmax_all",
+                               limit=float(f["expert"]["limit"]), groups=int(g.get("count") or 1), groups_keep=int(g.get("keep") or 1),
+                               shared=shared)
+        if spec.experts % spec.groups or not 1 <= spec.groups_keep <= spec.groups:
+            raise ValueError(f"layer {i}: {spec.groups_keep} of {spec.groups} groups over {spec.experts} experts")
+        if not 1 <= spec.top <= spec.groups_keep * (spec.experts // spec.groups):
+            raise ValueError(f"layer {i}: top {spec.top} of {spec.groups_keep} groups of {spec.experts // spec.groups} experts")
+        return spec
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "GekavikConfig":
+        layers = []
+        for i, ld in enumerate(d["layers"]):
+            kind = ld["type"]
+            if kind == "attention":
+                mixer = cls._attention(ld["mixer"], i)
+            elif kind == "latent_attention":
+                mixer = cls._latent(ld["mixer"], i)
+            else:
+                raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+            layers.append(GekavikLayerSpec(kind, mixer, cls._moe(ld["mlp"], i) if ld.get("mlp") else None, raw=ld))
+        lp = d.get("loop")
+        loop = {k: int(lp[k]) for k in ("start", "stop", "times")} if lp else None
+        if loop is not None and not (0 <= loop["start"] < loop["stop"] <= len(layers) and loop["times"] >= 1):
+            raise ValueError(f"loop {loop} does not fit {len(layers)} layers")
+        return cls(architecture=d["architecture"], vocab=int(d["vocab"]), width=int(d["width"]), norm_eps=float(d["norm"]["eps"]),
+                   residual_mult=float(d["residual_mult"]), layers=layers, loop=loop)
+
+    @classmethod
+    def from_pretrained(cls, model_dir: str) -> "GekavikConfig":
+        with open(os.path.join(model_dir, "config.json")) as f:
+            return cls.from_dict(json.load(f))
+
+    def runs(self) -> list[tuple[int, int | None]]:
+        """(layer index, number of the pass that starts right before it or None) of every layer run, in order."""
+        return loop_runs(len(self.layers), self.loop)
+
+    def to_dict(self) -> dict:
+        out = {"architecture": self.architecture, "vocab": self.vocab, "width": self.width, "norm": {"eps": self.norm_eps},
+               "residual_mult": self.residual_mult, "layers": [dict(l.raw) for l in self.layers]}
         if self.loop:
             out["loop"] = dict(self.loop)
         return out

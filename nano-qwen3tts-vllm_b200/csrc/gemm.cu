@@ -30,6 +30,7 @@
 #include <stdio.h>
 #include <stdlib.h>
 
+#include "clamped_gate.cuh"
 #include "umma.cuh"
 
 namespace b2 {
@@ -55,6 +56,8 @@ struct GemmParams {
   int splits;                   // cluster size along K
   int epilogue;                 // B2TTS_GEMM_*
   int rounding;                 // B2TTS_ROUND_* of the SiLU*mul epilogue
+  int out_f32;                  // `out` is a float tensor (bias epilogue): the sums leave unrounded
+  float act_limit, act_alpha;   // the clamped gated epilogue
   int tmem_cols;                // power of two >= 32, >= mpad
   int stages;                   // ring depth (2..4)
   // fused input RMSNorm: x is the RESIDUAL stream; the x producers stage norm(x) = f(x * rstd[m], w[k])
@@ -433,6 +436,15 @@ gemm_stream_kernel(const GemmParams p, const __grid_constant__ CUtensorMap tmap_
         stg_v2(p.out + (int64_t)(row0 + m) * p.out_stride + (n >> 1), w);
         return 0.f;
       }
+      if (p.epilogue == B2TTS_GEMM_CLAMPED_GATE) {
+        float o[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) o[j] = clamped_gate(acc[j], acc[4 + j], p.act_limit, p.act_alpha);
+        uint2 w;
+        w.x = pack_bf16(o[0], o[1]); w.y = pack_bf16(o[2], o[3]);
+        stg_v2(p.out + (int64_t)(row0 + m) * p.out_stride + (n >> 1), w);
+        return 0.f;
+      }
       if (p.epilogue == B2TTS_GEMM_BIAS && p.bias) {
         const uint4 bw = have_pre ? pre : ldg_v4(p.bias + n);
         acc[0] += bf16lo(bw.x); acc[1] += bf16hi(bw.x); acc[2] += bf16lo(bw.y); acc[3] += bf16hi(bw.y);
@@ -448,6 +460,12 @@ gemm_stream_kernel(const GemmParams p, const __grid_constant__ CUtensorMap tmap_
         acc[2] = rbf(acc[2]) + bf16lo(rw.y); acc[3] = rbf(acc[3]) + bf16hi(rw.y);
         acc[4] = rbf(acc[4]) + bf16lo(rw.z); acc[5] = rbf(acc[5]) + bf16hi(rw.z);
         acc[6] = rbf(acc[6]) + bf16lo(rw.w); acc[7] = rbf(acc[7]) + bf16hi(rw.w);
+      }
+      if (p.out_f32) {
+        float* o = reinterpret_cast<float*>(p.out) + (int64_t)(row0 + m) * p.out_stride + n;
+        *reinterpret_cast<float4*>(o) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+        *reinterpret_cast<float4*>(o + 4) = make_float4(acc[4], acc[5], acc[6], acc[7]);
+        return 0.f;
       }
       uint4 w;
       w.x = pack_bf16(acc[0], acc[1]); w.y = pack_bf16(acc[2], acc[3]);
@@ -693,7 +711,9 @@ static int gemm_impl(const char* what, const void* x, int64_t x_row_stride, cons
                      void* out, int64_t out_row_stride, int m, int n, int k,
                      int epilogue, int rounding, int splits, int pdl,
                      const void* norm_weight, const float* ssq_in, int ssq_in_slots, float eps, float* ssq_out,
-                     const void* prefetch_next, size_t prefetch_bytes, void* stream) {
+                     const void* prefetch_next, size_t prefetch_bytes, void* stream, int out_f32 = 0, float act_limit = 0.f,
+                     float act_alpha = 0.f) {
+  B2_REQUIRE(!out_f32 || (epilogue == B2TTS_GEMM_BIAS && !ssq_out), B2TTS_EINVAL, "%s: float output with epilogue %d", what, epilogue);
   B2_REQUIRE(m >= 0 && n > 0 && k > 0, B2TTS_EINVAL, "%s: m=%d n=%d k=%d", what, m, n, k);
   B2_REQUIRE(!prefetch_next || (aligned16(prefetch_next) && prefetch_bytes % G_WTILE_BYTES == 0), B2TTS_EALIGN,
              "%s: prefetch_next must be a packed weight image (16-byte aligned, a multiple of %d bytes)", what, G_WTILE_BYTES);
@@ -702,16 +722,17 @@ static int gemm_impl(const char* what, const void* x, int64_t x_row_stride, cons
              "%s: m=%d (1..%d), n=%d (multiple of %d), k=%d (multiple of %d)", what, m, G_MAX_ROWS, n, G_BN, k, G_BK);
   B2_REQUIRE(x && w_packed && out, B2TTS_EINVAL, "%s: null pointer", what);
   B2_REQUIRE(epilogue == B2TTS_GEMM_BIAS || epilogue == B2TTS_GEMM_RESIDUAL || epilogue == B2TTS_GEMM_SILU_MUL ||
-                 epilogue == B2TTS_GEMM_RELU_SQ || epilogue == B2TTS_GEMM_GELU_MUL, B2TTS_EINVAL, "%s: epilogue %d", what, epilogue);
+                 epilogue == B2TTS_GEMM_RELU_SQ || epilogue == B2TTS_GEMM_GELU_MUL || epilogue == B2TTS_GEMM_CLAMPED_GATE,
+             B2TTS_EINVAL, "%s: epilogue %d", what, epilogue);
+  const bool gated = epilogue == B2TTS_GEMM_SILU_MUL || epilogue == B2TTS_GEMM_GELU_MUL || epilogue == B2TTS_GEMM_CLAMPED_GATE;
   B2_REQUIRE(epilogue != B2TTS_GEMM_RESIDUAL || residual, B2TTS_EINVAL, "%s: residual epilogue without residual", what);
   B2_REQUIRE(aligned16(x) && aligned16(w_packed) && aligned16(out) && x_row_stride % 8 == 0 && out_row_stride % 4 == 0 &&
-                 (epilogue == B2TTS_GEMM_SILU_MUL || epilogue == B2TTS_GEMM_GELU_MUL || out_row_stride % 8 == 0) &&
+                 (gated || out_row_stride % 8 == 0) &&
                  (!bias || aligned16(bias)) && (!residual || (aligned16(residual) && residual_row_stride % 8 == 0)),
              B2TTS_EALIGN, "%s: pointers / strides must be 16-byte aligned", what);
   B2_REQUIRE(!norm_weight || (ssq_in && ssq_in_slots > 0 && aligned16(norm_weight) && aligned16(ssq_in)), B2TTS_EINVAL,
              "%s: fused norm needs ssq_in with >= 1 slot per row (16-byte aligned)", what);
-  B2_REQUIRE(!ssq_out || (epilogue != B2TTS_GEMM_SILU_MUL && epilogue != B2TTS_GEMM_GELU_MUL), B2TTS_EINVAL,
-             "%s: ssq_out with a gated epilogue", what);
+  B2_REQUIRE(!ssq_out || !gated, B2TTS_EINVAL, "%s: ssq_out with a gated epilogue", what);
   GemmParams p{};
   p.x = static_cast<const __nv_bfloat16*>(x);
   p.x_stride = x_row_stride;
@@ -787,6 +808,9 @@ static int gemm_impl(const char* what, const void* x, int64_t x_row_stride, cons
   p.kblocks = k / G_BK;
   p.epilogue = epilogue;
   p.rounding = rounding;
+  p.out_f32 = out_f32;
+  p.act_limit = act_limit;
+  p.act_alpha = act_alpha;
   // splits < 0: a batch split of -splits CTAs (see GemmParams::bsplit); 0: chosen here
   int bs = 1;
   if (splits < 0) {
@@ -853,6 +877,18 @@ extern "C" int b2tts_gemm_bf16(const void* x, int64_t x_row_stride, const void* 
                                int epilogue, int rounding, int splits, int pdl, void* stream) {
   return b2::gemm_impl("gemm_bf16", x, x_row_stride, w_packed, bias, residual, residual_row_stride, out, out_row_stride,
                        m, n, k, epilogue, rounding, splits, pdl, nullptr, nullptr, 0, 0.f, nullptr, nullptr, 0, stream);
+}
+
+extern "C" int b2tts_gemm_f32out_bf16(const void* x, int64_t x_row_stride, const void* w_packed, const void* bias, float* out,
+                                      int64_t out_row_stride, int m, int n, int k, int splits, int pdl, void* stream) {
+  return b2::gemm_impl("gemm_f32out_bf16", x, x_row_stride, w_packed, bias, nullptr, 0, out, out_row_stride, m, n, k, B2TTS_GEMM_BIAS, 0,
+                       splits, pdl, nullptr, nullptr, 0, 0.f, nullptr, nullptr, 0, stream, 1);
+}
+
+extern "C" int b2tts_gemm_clamped_gate_bf16(const void* x, int64_t x_row_stride, const void* w_packed, void* out, int64_t out_row_stride,
+                                            int m, int n, int k, float limit, float alpha, int splits, int pdl, void* stream) {
+  return b2::gemm_impl("gemm_clamped_gate_bf16", x, x_row_stride, w_packed, nullptr, nullptr, 0, out, out_row_stride, m, n, k,
+                       B2TTS_GEMM_CLAMPED_GATE, 0, splits, pdl, nullptr, nullptr, 0, 0.f, nullptr, nullptr, 0, stream, 0, limit, alpha);
 }
 
 extern "C" int b2tts_gemm_ssq_slots(int m, int n, int k, int splits) {

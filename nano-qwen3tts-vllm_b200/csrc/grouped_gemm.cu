@@ -7,7 +7,11 @@
 // the down projection reads row s and writes row `pair`, so that the caller's weighted sum over a token's choices reads
 // them in a fixed order.  Inputs are bf16 or float, products accumulate in float.  A tile never mixes two experts:
 // tile y of the grid is mapped to (expert, row block) by walking the group sizes, and tiles beyond the last group exit.
-#include "common.cuh"
+//
+// Gated experts (grouped_gemm_gated): W[e] is [gate; up], 2 ff rows.  A tile's 128 rows of W are 8 gate rows and the 8 matching
+// up rows in turn, so a thread's accumulators hold the gate and the up value of the same columns and the clamped gated product
+// is taken in the epilogue: C has ff columns and the [pairs, 2 ff] product never reaches memory.
+#include "clamped_gate.cuh"
 
 namespace b2 {
 
@@ -118,12 +122,14 @@ template <int BM> struct GmShape {
   static constexpr size_t SMEM = sizeof(__nv_bfloat16) * STAGES * (BM + GM_BN) * GM_LD + sizeof(int) * 2 * BM;
 };
 
+constexpr int ACT_GATED = 2;
+
 template <int GM_BM, int ACT>
 __global__ void __launch_bounds__(GM_THREADS, 2)
 grouped_gemm_mma_kernel(const __nv_bfloat16* __restrict__ A, int64_t lda, const __nv_bfloat16* __restrict__ W,
                         __nv_bfloat16* __restrict__ C, int64_t ldc, const int32_t* __restrict__ offsets,
                         const int32_t* __restrict__ sorted_pair, int E, int N, int K, int top, int in_by_token, int out_by_pair,
-                        int paired_store) {
+                        int paired_store, float limit, float alpha) {
   using S = GmShape<GM_BM>;
   constexpr int GM_STAGES = S::STAGES, MT = S::MT, NT = S::NT;
   extern __shared__ __align__(16) unsigned char gm_smem[];
@@ -162,7 +168,12 @@ grouped_gemm_mma_kernel(const __nv_bfloat16* __restrict__ A, int64_t lda, const 
   for (int i = 0; i < GM_PASSES; ++i) {
     const int r = GM_RPP * i + tid / GM_CPR;
     a_row[i] = r < GM_BM ? in_rows[r] : -1;
-    w_row[i] = n0 + r < N ? n0 + r : -1;
+    if constexpr (ACT == ACT_GATED) {
+      const int f = n0 / 2 + (r >> 4) * 8 + (r & 7);      // 8 gate rows, 8 up rows, ..
+      w_row[i] = f < N / 2 ? f + ((r >> 3) & 1) * (N / 2) : -1;
+    } else {
+      w_row[i] = n0 + r < N ? n0 + r : -1;
+    }
   }
   const int ck = (tid % GM_CPR) * 8;
   const int nk = (K + GM_BK - 1) / GM_BK;
@@ -223,6 +234,16 @@ grouped_gemm_mma_kernel(const __nv_bfloat16* __restrict__ A, int64_t lda, const 
       const int orow = out_rows[r];
       if (orow < 0) continue;
       __nv_bfloat16* crow = C + static_cast<int64_t>(orow) * ldc;
+      if constexpr (ACT == ACT_GATED) {
+#pragma unroll
+        for (int np = 0; np < NT / 2; ++np) {
+          const int n = n0 / 2 + (wn * (NT / 2) + np) * 8 + 2 * (lane & 3);
+          const float v0 = clamped_gate(acc[mt][2 * np][2 * half], acc[mt][2 * np + 1][2 * half], limit, alpha);
+          const float v1 = clamped_gate(acc[mt][2 * np][2 * half + 1], acc[mt][2 * np + 1][2 * half + 1], limit, alpha);
+          if (n < N / 2) *reinterpret_cast<uint32_t*>(crow + n) = pack_bf16(v0, v1);      // ff is a multiple of 8
+        }
+        continue;
+      }
 #pragma unroll
       for (int nt = 0; nt < NT; ++nt) {
         const int n = n0 + wn * NT * 8 + nt * 8 + 2 * (lane & 3);
@@ -242,7 +263,7 @@ grouped_gemm_mma_kernel(const __nv_bfloat16* __restrict__ A, int64_t lda, const 
 template <int BM, int ACT>
 static cudaError_t launch_grouped_mma(int n_pairs, cudaStream_t st, const void* a, int64_t lda, const void* w, void* c, int64_t ldc,
                                       const int32_t* offsets, const int32_t* sorted_pair, int E, int N, int K, int top,
-                                      int in_by_token, int out_by_pair) {
+                                      int in_by_token, int out_by_pair, float limit = 0.f, float alpha = 0.f) {
   auto kern = grouped_gemm_mma_kernel<BM, ACT>;
   constexpr size_t GM_SMEM = GmShape<BM>::SMEM;
   const dim3 grid((N + GM_BN - 1) / GM_BN, (n_pairs + BM - 1) / BM + E);
@@ -251,7 +272,7 @@ static cudaError_t launch_grouped_mma(int n_pairs, cudaStream_t st, const void* 
   const int paired = (ldc % 2 == 0) && (reinterpret_cast<uintptr_t>(c) % 4 == 0);
   kern<<<grid, GM_THREADS, GM_SMEM, st>>>(static_cast<const __nv_bfloat16*>(a), lda, static_cast<const __nv_bfloat16*>(w),
                                           static_cast<__nv_bfloat16*>(c), ldc, offsets, sorted_pair, E, N, K, top, in_by_token,
-                                          out_by_pair, paired);
+                                          out_by_pair, paired, limit, alpha);
   return cudaSuccess;
 }
 
@@ -285,5 +306,24 @@ extern "C" int b2tts_grouped_gemm(const void* a, int64_t lda, const void* w, voi
   else { if (act) GG_GO(float, 1); else GG_GO(float, 0); }
 #undef GG_GO
   B2_CHECK_LAUNCH("grouped_gemm");
+  return B2TTS_OK;
+}
+
+extern "C" int b2tts_grouped_gemm_gated(const void* a, int64_t lda, const void* w, void* c, int64_t ldc, const int32_t* offsets,
+                                        const int32_t* sorted_pair, int n_pairs, int experts, int ff, int k, int top, float limit,
+                                        float alpha, void* stream) {
+  using namespace b2;
+  B2_REQUIRE(n_pairs >= 0 && experts > 0 && ff > 0 && k > 0 && top > 0, B2TTS_EINVAL, "grouped_gemm_gated: bad sizes");
+  B2_REQUIRE(ff % 8 == 0 && k % 8 == 0 && lda % 8 == 0 && ldc % 2 == 0, B2TTS_EUNSUPPORTED, "grouped_gemm_gated: ff=%d k=%d must be multiples of 8",
+             ff, k);
+  if (n_pairs == 0) return B2TTS_OK;
+  B2_REQUIRE(a && w && c && offsets && sorted_pair, B2TTS_EINVAL, "grouped_gemm_gated: null pointer");
+  B2_REQUIRE(aligned16(a) && aligned16(w) && aligned16(c), B2TTS_EALIGN, "grouped_gemm_gated: pointers must be 16-byte aligned");
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool small = n_pairs <= 16 * experts;
+  const cudaError_t e = small ? launch_grouped_mma<32, ACT_GATED>(n_pairs, st, a, lda, w, c, ldc, offsets, sorted_pair, experts, 2 * ff, k, top, 1, 0, limit, alpha)
+                              : launch_grouped_mma<128, ACT_GATED>(n_pairs, st, a, lda, w, c, ldc, offsets, sorted_pair, experts, 2 * ff, k, top, 1, 0, limit, alpha);
+  if (e != cudaSuccess) return cuda_fail(e, "grouped_gemm_gated");
+  B2_CHECK_LAUNCH("grouped_gemm_gated");
   return B2TTS_OK;
 }

@@ -289,6 +289,179 @@ attn_prep_kernel(const T* __restrict__ u, int64_t ldu, int q_off, int k_off, int
   }
 }
 
+// The preparation of heads that are normed ONE BY ONE: v' = N_head(v + bias) * w (w of `dim` numbers, shared by the heads), then
+// the rotation by the step's table `rot` [n, rot_dims] (cosines, then sines).  Work items are (token run, head): heads 0 .. H-1
+// are queries, then G key heads, then G value heads (bias and cache write only).
+struct HeadPrepArgs {
+  const void* u; int64_t ldu; int q_off, k_off, v_off;
+  const float *q_bias, *k_bias, *v_bias, *q_norm_w, *k_norm_w;
+  const float* rot; int rot_dims, interleaved;
+  const int32_t* slot_mapping;
+  void *q_out, *k_cache, *v_cache;
+  int n_tokens, H, G, d, dv;
+  float eps;
+};
+
+template <typename T>
+struct HeadSlice {                                        // what a head reads and writes
+  const T* src; const float* bias; const float* nw; T* dst;
+  int64_t dst_row; int width; bool cached, qk;
+  __device__ __forceinline__ HeadSlice(const HeadPrepArgs& p, int head) {
+    const T* u = static_cast<const T*>(p.u);
+    if (head < p.H) {
+      src = u + p.q_off + head * p.d; bias = p.q_bias ? p.q_bias + head * p.d : nullptr; nw = p.q_norm_w;
+      dst = static_cast<T*>(p.q_out) + head * p.d; dst_row = static_cast<int64_t>(p.H) * p.d; width = p.d; cached = false; qk = true;
+    } else if (head < p.H + p.G) {
+      const int g = head - p.H;
+      src = u + p.k_off + g * p.d; bias = p.k_bias ? p.k_bias + g * p.d : nullptr; nw = p.k_norm_w;
+      dst = static_cast<T*>(p.k_cache) + g * p.d; dst_row = static_cast<int64_t>(p.G) * p.d; width = p.d; cached = true; qk = true;
+    } else {
+      const int g = head - p.H - p.G;
+      src = u + p.v_off + g * p.dv; bias = p.v_bias ? p.v_bias + g * p.dv : nullptr; nw = nullptr;
+      dst = static_cast<T*>(p.v_cache) + g * p.dv; dst_row = static_cast<int64_t>(p.G) * p.dv; width = p.dv; cached = true; qk = false;
+    }
+  }
+};
+
+constexpr int HP_WARPS = 8;
+
+// Any head size, either pairing: one warp per (token, head).
+template <typename T>
+__global__ void __launch_bounds__(HP_WARPS * 32)
+head_prep_kernel(const HeadPrepArgs p) {
+  const int heads = p.H + 2 * p.G, lane = threadIdx.x & 31;
+  const int64_t item = static_cast<int64_t>(blockIdx.x) * HP_WARPS + (threadIdx.x >> 5);
+  if (item >= static_cast<int64_t>(p.n_tokens) * heads) return;
+  const size_t t = item / heads;
+  const HeadSlice<T> s(p, static_cast<int>(item % heads));
+  const int slot = p.slot_mapping[t];
+  if (slot < 0) return;                                   // padding row
+  const T* src = s.src + t * p.ldu;
+  T* dst = s.dst + (s.cached ? static_cast<int64_t>(slot) : static_cast<int64_t>(t)) * s.dst_row;
+  auto val = [&](int c) { return to_f(src[c]) + (s.bias != nullptr ? s.bias[c] : 0.f); };
+  float inv = 1.f;
+  if (s.nw != nullptr) {
+    float ssq = 0.f;
+    for (int c = lane; c < s.width; c += 32) { const float v = val(c); ssq += v * v; }
+    inv = 1.0f / sqrtf(warp_sum(ssq) / static_cast<float>(s.width) + p.eps);
+  }
+  const int rd = s.qk ? p.rot_dims : 0, half = rd / 2;
+  for (int c = lane; c < s.width; c += 32) {
+    if (c < rd && (p.interleaved ? (c & 1) : c >= half)) continue;        // second of a pair: written with the first
+    float a = val(c) * inv * (s.nw != nullptr ? s.nw[c] : 1.f);
+    if (c < rd) {
+      const int c2 = p.interleaved ? c + 1 : c + half, i = p.interleaved ? c >> 1 : c;
+      const float b = val(c2) * inv * (s.nw != nullptr ? s.nw[c2] : 1.f);
+      const float cs = p.rot[t * rd + i], sn = p.rot[t * rd + half + i];
+      dst[c] = from_f<T>(a * cs - b * sn);
+      dst[c2] = from_f<T>(b * cs + a * sn);
+    } else {
+      dst[c] = from_f<T>(a);
+    }
+  }
+}
+
+template <typename T> __device__ __forceinline__ void load4_f(const T* p, float* f);
+template <> __device__ __forceinline__ void load4_f<float>(const float* p, float* f) {
+  const float4 v = *reinterpret_cast<const float4*>(p);
+  f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+}
+template <> __device__ __forceinline__ void load4_f<__nv_bfloat16>(const __nv_bfloat16* p, float* f) {
+  const uint2 r = ldg_v2(p);
+  f[0] = bf16lo(r.x); f[1] = bf16hi(r.x); f[2] = bf16lo(r.y); f[3] = bf16hi(r.y);
+}
+
+// Pairs (2i, 2i + 1) or no rotation, sizes and offsets multiples of 4: LPH lanes share a head, four neighbouring coordinates
+// (two whole pairs) per lane and chunk, so 32 / LPH heads run in a warp and nothing but the sum of squares crosses lanes.  A lane
+// group walks TOK tokens of its head with bias and norm weight in registers; the rows of all TOK tokens are asked for first.
+template <typename T, int LPH, int NCH, int TOK>
+__global__ void __launch_bounds__(HP_WARPS * 32)
+head_prep_vec4_kernel(const HeadPrepArgs p) {
+  const int heads = p.H + 2 * p.G, sub = threadIdx.x % LPH;
+  const int64_t item = (static_cast<int64_t>(blockIdx.x) * (HP_WARPS * 32) + threadIdx.x) / LPH;
+  const int64_t n_items = static_cast<int64_t>((p.n_tokens + TOK - 1) / TOK) * heads;
+  const bool live = item < n_items;                       // every lane stays for the shuffles
+  const int t0 = live ? static_cast<int>(item / heads) * TOK : 0;
+  const HeadSlice<T> s(p, live ? static_cast<int>(item % heads) : 0);
+  const int rd = s.qk ? p.rot_dims : 0;
+  float x[TOK][NCH][4], bias[NCH][4], w[NCH][4];
+  int slot[TOK];
+#pragma unroll
+  for (int t = 0; t < TOK; ++t) slot[t] = live && t0 + t < p.n_tokens ? p.slot_mapping[t0 + t] : -1;
+#pragma unroll
+  for (int k = 0; k < NCH; ++k) {
+    const int c = (k * LPH + sub) * 4;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) { bias[k][e] = 0.f; w[k][e] = 1.f; }
+#pragma unroll
+    for (int t = 0; t < TOK; ++t) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) x[t][k][e] = 0.f;
+      if (c < s.width && slot[t] >= 0) load4_f<T>(s.src + static_cast<int64_t>(t0 + t) * p.ldu + c, x[t][k]);
+    }
+    if (c < s.width) {
+      if (s.bias != nullptr) load4_f<float>(s.bias + c, bias[k]);
+      if (s.nw != nullptr) load4_f<float>(s.nw + c, w[k]);
+    }
+  }
+#pragma unroll
+  for (int t = 0; t < TOK; ++t) {
+    float ssq = 0.f;
+#pragma unroll
+    for (int k = 0; k < NCH; ++k)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) { x[t][k][e] += bias[k][e]; ssq += x[t][k][e] * x[t][k][e]; }
+#pragma unroll
+    for (int o = LPH / 2; o > 0; o >>= 1) ssq += __shfl_xor_sync(0xffffffffu, ssq, o);
+    if (slot[t] < 0) continue;
+    const float inv = s.nw != nullptr ? 1.0f / sqrtf(ssq / static_cast<float>(s.width) + p.eps) : 1.f;
+    T* dst = s.dst + (s.cached ? static_cast<int64_t>(slot[t]) : static_cast<int64_t>(t0 + t)) * s.dst_row;
+    const float* rot = p.rot + static_cast<int64_t>(t0 + t) * rd;
+#pragma unroll
+    for (int k = 0; k < NCH; ++k) {
+      const int c = (k * LPH + sub) * 4;
+      if (c >= s.width) continue;
+      float v[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[e] = x[t][k][e] * inv * w[k][e];
+      if (c < rd) {                                       // rot_dims is a multiple of 4: both pairs turn, or neither
+        const float2 cs = *reinterpret_cast<const float2*>(rot + c / 2), sn = *reinterpret_cast<const float2*>(rot + rd / 2 + c / 2);
+        const float a0 = v[0], a1 = v[2];
+        v[0] = a0 * cs.x - v[1] * sn.x; v[1] = v[1] * cs.x + a0 * sn.x;
+        v[2] = a1 * cs.y - v[3] * sn.y; v[3] = v[3] * cs.y + a1 * sn.y;
+      }
+      if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(dst + c) = make_float4(v[0], v[1], v[2], v[3]);
+      else stg_v2(dst + c, make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3])));
+    }
+  }
+}
+
+template <typename T>
+static void launch_head_prep(const HeadPrepArgs& p, cudaStream_t st) {
+  const int heads = p.H + 2 * p.G, wide = std::max(p.d, p.dv);
+  const bool vec = p.d % 4 == 0 && p.dv % 4 == 0 && p.ldu % 4 == 0 && p.q_off % 4 == 0 && p.k_off % 4 == 0 && p.v_off % 4 == 0 &&
+                   wide <= 256 && (p.rot_dims == 0 || (p.interleaved && p.rot_dims % 4 == 0 && aligned16(p.rot))) && aligned16(p.u) &&
+                   aligned16(p.q_out) && aligned16(p.k_cache) && aligned16(p.v_cache) && (!p.q_bias || aligned16(p.q_bias)) &&
+                   (!p.k_bias || aligned16(p.k_bias)) && (!p.v_bias || aligned16(p.v_bias)) && (!p.q_norm_w || aligned16(p.q_norm_w)) &&
+                   (!p.k_norm_w || aligned16(p.k_norm_w));
+  if (!vec) {
+    const int64_t items = static_cast<int64_t>(p.n_tokens) * heads;
+    head_prep_kernel<T><<<static_cast<unsigned>((items + HP_WARPS - 1) / HP_WARPS), HP_WARPS * 32, 0, st>>>(p);
+    return;
+  }
+  const bool many = static_cast<int64_t>(p.n_tokens) * heads > static_cast<int64_t>(sm_count()) * 256;
+#define HP_GO_T(LPH, NCH, TOK) do { \
+    const int64_t threads = static_cast<int64_t>((p.n_tokens + TOK - 1) / TOK) * heads * LPH; \
+    head_prep_vec4_kernel<T, LPH, NCH, TOK><<<static_cast<unsigned>((threads + HP_WARPS * 32 - 1) / (HP_WARPS * 32)), HP_WARPS * 32, 0, st>>>(p); } while (0)
+#define HP_GO(LPH, NCH) do { if (many) HP_GO_T(LPH, NCH, 4); else HP_GO_T(LPH, NCH, 1); } while (0)
+  if (wide <= 32) HP_GO(8, 1);
+  else if (wide <= 64) HP_GO(16, 1);
+  else if (wide <= 128) HP_GO(32, 1);
+  else HP_GO(32, 2);
+#undef HP_GO
+#undef HP_GO_T
+}
+
 // ------------------------------------------------------------------ short causal convolution + activation
 // y[t, c] = act(bias[c] + sum_j w[c, j] * u(position(t) - taps + 1 + j)[c]) over the C columns of u from c_off on.  An
 // earlier position comes from this step's rows when it lies in the step's portion, from the sequence's carried state
@@ -670,6 +843,25 @@ extern "C" int b2tts_attn_prep(const void* u, int64_t ldu, int q_off, int k_off,
         v_bias, q_norm_w, k_norm_w, freq, rot_dims, positions, slot_mapping, static_cast<float*>(q_out),
         static_cast<float*>(k_cache), static_cast<float*>(v_cache), heads, kv_heads, v_heads, dim, vdim, eps, interleaved);
   B2_CHECK_LAUNCH("attn_prep");
+  return B2TTS_OK;
+}
+
+extern "C" int b2tts_attn_head_prep(const void* u, int64_t ldu, int q_off, int k_off, int v_off, const float* q_bias, const float* k_bias,
+                                    const float* v_bias, const float* q_norm_w, const float* k_norm_w, const float* rot, int rot_dims,
+                                    int interleaved, const int32_t* slot_mapping, void* q_out, void* k_cache, void* v_cache,
+                                    int n_tokens, int heads, int kv_heads, int dim, int vdim, float eps, int dtype, void* stream) {
+  B2_REQUIRE(n_tokens >= 0 && heads > 0 && kv_heads > 0 && dim > 0 && vdim > 0 && q_off >= 0 && k_off >= 0 && v_off >= 0, B2TTS_EINVAL,
+             "attn_head_prep: bad sizes");
+  B2_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dim, B2TTS_EINVAL, "attn_head_prep: %d rotated of %d coordinates", rot_dims, dim);
+  B2_REQUIRE((q_norm_w == nullptr) == (k_norm_w == nullptr), B2TTS_EINVAL, "attn_head_prep: norm weights for q and k, or neither");
+  B2_REQUIRE(B2_ROW_DTYPE_OK(dtype), B2TTS_EINVAL, "attn_head_prep: dtype %d", dtype);
+  if (n_tokens == 0) return B2TTS_OK;
+  B2_REQUIRE(u && slot_mapping && q_out && k_cache && v_cache && (rot_dims == 0 || rot), B2TTS_EINVAL, "attn_head_prep: null pointer");
+  const HeadPrepArgs p{u, ldu, q_off, k_off, v_off, q_bias, k_bias, v_bias, q_norm_w, k_norm_w, rot, rot_dims, interleaved, slot_mapping,
+                       q_out, k_cache, v_cache, n_tokens, heads, kv_heads, dim, vdim, eps};
+  if (dtype == B2TTS_DTYPE_BF16) launch_head_prep<__nv_bfloat16>(p, static_cast<cudaStream_t>(stream));
+  else launch_head_prep<float>(p, static_cast<cudaStream_t>(stream));
+  B2_CHECK_LAUNCH("attn_head_prep");
   return B2TTS_OK;
 }
 

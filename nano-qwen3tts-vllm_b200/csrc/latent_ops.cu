@@ -161,17 +161,18 @@ latent_prep_kernel(const T* __restrict__ u, int64_t ldu, int q_off, int kv_off, 
 }
 
 // ------------------------------------------------------------------ gate of the attention output + head-major -> row-major
-// out[t, h * dv + d] = v[h, t, d] (strides given) * sigmoid(gate[t, h * dv + d]); without a gate it is the plain re-layout.
+// out[t, h * dv + d] = v[h, t, d] (strides given) * sigmoid(gate[t, h * dv + d]), or, `per_head`, * sigmoid(gate[t, h]); without
+// a gate it is the plain re-layout.
 template <typename T>
 __global__ void gate_heads_kernel(const T* __restrict__ v, int64_t v_tok, int64_t v_head, const T* __restrict__ gate, int64_t ldg,
-                                  T* __restrict__ out, int n, int H, int dv) {
+                                  T* __restrict__ out, int n, int H, int dv, int per_head) {
   const size_t total = static_cast<size_t>(n) * H * dv;
   for (size_t i = blockIdx.x * static_cast<size_t>(blockDim.x) + threadIdx.x; i < total; i += static_cast<size_t>(gridDim.x) * blockDim.x) {
     const int d = static_cast<int>(i % dv);
     const int h = static_cast<int>((i / dv) % H);
     const size_t t = i / (static_cast<size_t>(dv) * H);
     float val = to_f(v[t * v_tok + h * v_head + d]);
-    if (gate != nullptr) val *= 1.0f / (1.0f + expf(-to_f(gate[t * ldg + static_cast<size_t>(h) * dv + d])));
+    if (gate != nullptr) val *= 1.0f / (1.0f + expf(-to_f(gate[t * ldg + (per_head ? h : static_cast<size_t>(h) * dv + d)])));
     out[i] = from_f<T>(val);
   }
 }
@@ -320,7 +321,7 @@ extern "C" int b2tts_latent_prep(const void* u, int64_t ldu, int q_off, int kv_o
 }
 
 extern "C" int b2tts_gate_heads(const void* v, int64_t v_tok, int64_t v_head, const void* gate, int64_t ldg, void* out, int n,
-                                int heads, int vdim, int dtype, void* stream) {
+                                int heads, int vdim, int per_head, int dtype, void* stream) {
   using namespace b2;
   using namespace b2::lat;
   B2_REQUIRE(n >= 0 && heads > 0 && vdim > 0 && LAT_DTYPE_OK(dtype), B2TTS_EINVAL, "gate_heads: n=%d heads=%d vdim=%d", n, heads, vdim);
@@ -329,7 +330,7 @@ extern "C" int b2tts_gate_heads(const void* v, int64_t v_tok, int64_t v_head, co
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int grid = flat_grid(static_cast<size_t>(n) * heads * vdim);
   LAT_DISPATCH(dtype, (gate_heads_kernel<T><<<grid, 256, 0, st>>>(static_cast<const T*>(v), v_tok, v_head, static_cast<const T*>(gate), ldg,
-                                                                 static_cast<T*>(out), n, heads, vdim)));
+                                                                 static_cast<T*>(out), n, heads, vdim, per_head)));
   B2_CHECK_LAUNCH("gate_heads");
   return B2TTS_OK;
 }

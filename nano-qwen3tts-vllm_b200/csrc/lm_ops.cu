@@ -522,6 +522,8 @@ __global__ void conv_state_update_kernel(const T* __restrict__ u, int64_t u_stri
 // mode 1: scores = logits + bias, weights = softmax over the chosen scores * scale.
 // mode 2: scores = softmax over ALL logits; the choice is made on score + bias, the weights are the chosen scores
 //         themselves * scale, not renormalised.
+// groups > 1: the experts form that many equal groups of neighbours, a group counts as much as its largest choice score, and
+// only experts of the groups_keep best groups (ties: the lower group) can be chosen.
 constexpr int ROUTE_WARPS = 4;
 constexpr int ROUTE_MAX_EXPERTS = 256;
 
@@ -529,7 +531,8 @@ template <typename T>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router /* [E, cols] */, int32_t* __restrict__ top_idx,
                  float* __restrict__ top_w, int n_tokens, int cols, int E, int top, float scale,
-                 const float* __restrict__ bias /* [E] or null */, int mode) {
+                 const float* __restrict__ bias /* [E] or null */, int mode, int groups, int groups_keep) {
+  __shared__ float gscore[ROUTE_WARPS][ROUTE_MAX_EXPERTS];   // groups: their scores, then whether they were kept
   __shared__ float score[ROUTE_WARPS][ROUTE_MAX_EXPERTS];
   __shared__ float weight[ROUTE_WARPS][ROUTE_MAX_EXPERTS];   // mode 2: the scores the weights are taken from
   const int softmax_chosen = mode == 1;
@@ -571,6 +574,27 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router /* [E
     }
     __syncwarp();
   }
+  if (groups > 1) {
+    const int per = E / groups;
+    for (int g = lane; g < groups; g += 32) {
+      float best = -INFINITY;
+      for (int e = g * per; e < (g + 1) * per; ++e) best = fmaxf(best, score[warp][e]);
+      gscore[warp][g] = best;
+    }
+    __syncwarp();
+    // a group is kept when fewer than groups_keep others come before it
+    unsigned long long kept = 0ull;                       // bit i: the lane's group lane + 32 i
+    for (int g = lane, i = 0; g < groups; g += 32, ++i) {
+      const float mine = gscore[warp][g];
+      int before = 0;
+      for (int o = 0; o < groups; ++o) before += gscore[warp][o] > mine || (gscore[warp][o] == mine && o < g);
+      if (before < groups_keep) kept |= 1ull << i;
+    }
+    for (int g = lane, i = 0; g < groups; g += 32, ++i)
+      if (!(kept >> i & 1ull))
+        for (int e = g * per; e < (g + 1) * per; ++e) score[warp][e] = -INFINITY;
+    __syncwarp();
+  }
   float sum = 0.f, first = 0.f;
   float chosen_s = 0.f;          // lane k keeps the k-th choice
   int chosen_e = 0;
@@ -587,6 +611,7 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router /* [E
       const int oe = __shfl_xor_sync(0xffffffffu, be, o);
       if (ob > best || (ob == best && oe < be)) { best = ob; be = oe; }
     }
+    if (be >= E) be = 0;                                  // no finite score left (NaN inputs): still a valid expert id
     if (k == 0) first = best;
     if (softmax_chosen) best = expf(best - first);       // weights: the softmax over the chosen logits only
     if (mode == 2) best = weight[warp][be];
@@ -783,9 +808,11 @@ extern "C" int b2tts_conv_headnorm_kvwrite(const void* u, int64_t u_stride, cons
 
 extern "C" int b2tts_moe_route(const void* h, const float* router, int32_t* top_idx, float* top_w, int32_t* offsets,
                                int32_t* sorted_pair, int n_tokens, int cols, int experts, int top, float scale,
-                               const float* bias, int mode, int dtype, void* stream) {
+                               const float* bias, int mode, int groups, int groups_keep, int dtype, void* stream) {
   using namespace b2;
   B2_REQUIRE(n_tokens >= 0 && cols > 0 && experts > 0 && top > 0 && top <= experts, B2TTS_EINVAL, "moe_route: bad sizes");
+  B2_REQUIRE(groups >= 1 && experts % groups == 0 && groups_keep >= 1 && groups_keep <= groups && top <= groups_keep * (experts / groups),
+             B2TTS_EINVAL, "moe_route: top %d of %d of %d groups over %d experts", top, groups_keep, groups, experts);
   B2_REQUIRE(mode >= 0 && mode <= 2, B2TTS_EINVAL, "moe_route: mode %d", mode);
   B2_REQUIRE(experts <= ROUTE_MAX_EXPERTS && top <= 32, B2TTS_EUNSUPPORTED, "moe_route: experts %d > %d or top %d > 32", experts,
              ROUTE_MAX_EXPERTS, top);
@@ -797,10 +824,11 @@ extern "C" int b2tts_moe_route(const void* h, const float* router, int32_t* top_
     const int grid = (n_tokens + ROUTE_WARPS - 1) / ROUTE_WARPS;
     if (dtype == B2TTS_DTYPE_BF16)
       moe_route_kernel<__nv_bfloat16><<<grid, ROUTE_WARPS * 32, 0, st>>>(static_cast<const __nv_bfloat16*>(h), router, top_idx, top_w,
-                                                                          n_tokens, cols, experts, top, scale, bias, mode);
+                                                                          n_tokens, cols, experts, top, scale, bias, mode, groups,
+                                                                          groups_keep);
     else
       moe_route_kernel<float><<<grid, ROUTE_WARPS * 32, 0, st>>>(static_cast<const float*>(h), router, top_idx, top_w, n_tokens, cols,
-                                                                 experts, top, scale, bias, mode);
+                                                                 experts, top, scale, bias, mode, groups, groups_keep);
     B2_CHECK_LAUNCH("moe_route");
   }
   moe_group_kernel<<<1, 1024, 0, st>>>(top_idx, offsets, sorted_pair, n_tokens * top, experts);

@@ -5,7 +5,7 @@
 //   window mask: max(0, i - mask + 1) <= j <= i        chunk mask: floor(i / mask) * mask <= j <= i        mask <= 0: j <= i
 //
 // Both masks are a lower bound on j, so one kernel serves them.  The sink has no key and no value and is not scaled.  An
-// optional per-head gate multiplies the head's output by sigmoid(gate[t, h]).
+// optional gate multiplies the head's output by sigmoid(gate[t, h]), or (gate_el) its elements by sigmoid(gate[t, h * dv + c]).
 //
 // Three more switches, each off at its neutral value: keep_first F > 0 lets every token also see the keys j < F that its mask
 // hides (the kernels then walk a virtual key list, [0, min(F, lo)) followed by [lo, i]); softcap c > 0 turns a scaled score
@@ -117,7 +117,7 @@ __global__ void __launch_bounds__(SA_WARPS * 32)
 sink_attn_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache, T* __restrict__ out,
                  const int32_t* __restrict__ tok_seq, const int32_t* __restrict__ positions, const int32_t* __restrict__ seq_len,
                  const int32_t* __restrict__ block_tables, int64_t bt_stride, const float* __restrict__ sink,
-                 const T* __restrict__ gate, int64_t ldg, int H, int G, int Gv, int d, int dv, int page, int mask_kind, int mask,
+                 const T* __restrict__ gate, int64_t ldg, int gate_el, int H, int G, int Gv, int d, int dv, int page, int mask_kind, int mask,
                  int keep_first, float softcap, float scale, int only_single, int out_f32) {
   extern __shared__ float smem[];
   const int qstride = (d + 3) & ~3;
@@ -236,12 +236,13 @@ sink_attn_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T
       den += cw[w] * part[(w * REP + r) * pstride + dv + 1];
     }
     float gv = 1.f;
-    if (gate != nullptr) gv = sigmoid_f(to_f(gate[t * ldg + h]));
+    if (gate != nullptr && !gate_el) gv = sigmoid_f(to_f(gate[t * ldg + h]));
     const float inv = gv / den;
     for (int c = threadIdx.x; c < dv; c += blockDim.x) {
       float o = 0.f;
 #pragma unroll
       for (int w = 0; w < SA_WARPS; ++w) o += cw[w] * part[(w * REP + r) * pstride + c];
+      if (gate != nullptr && gate_el) o *= sigmoid_f(to_f(gate[t * ldg + static_cast<int64_t>(h) * dv + c]));
       put_out(out, obase + r * dv + c, o * inv, out_f32);
     }
   }
@@ -250,21 +251,21 @@ sink_attn_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T
 template <typename T, int REP>
 static void launch_sink_plain(cudaStream_t st, const void* q, const void* kc, const void* vc, void* out, const int32_t* tok_seq,
                               const int32_t* positions, const int32_t* seq_len, const int32_t* bt, int64_t bt_stride, const float* sink,
-                              const void* gate, int64_t ldg, int n_tokens, int H, int G, int Gv, int d, int dv, int page, int mask_kind,
+                              const void* gate, int64_t ldg, int gate_el, int n_tokens, int H, int G, int Gv, int d, int dv, int page, int mask_kind,
                               int mask, int keep_first, float softcap, float scale, int only_single, int out_f32) {
   const size_t sm = (static_cast<size_t>(REP) * ((d + 3) & ~3) + static_cast<size_t>(SA_WARPS) * REP * (dv + 2)) * sizeof(float);
   sink_attn_kernel<T, REP><<<dim3(n_tokens, H / REP), SA_WARPS * 32, sm, st>>>(
       static_cast<const T*>(q), static_cast<const T*>(kc), static_cast<const T*>(vc), static_cast<T*>(out), tok_seq, positions, seq_len, bt,
-      bt_stride, sink, static_cast<const T*>(gate), ldg, H, G, Gv, d, dv, page, mask_kind, mask, keep_first, softcap, scale, only_single, out_f32);
+      bt_stride, sink, static_cast<const T*>(gate), ldg, gate_el, H, G, Gv, d, dv, page, mask_kind, mask, keep_first, softcap, scale, only_single, out_f32);
 }
 
 template <typename T>
 static void launch_sink_plain_rep(int rep, cudaStream_t st, const void* q, const void* kc, const void* vc, void* out,
                                   const int32_t* tok_seq, const int32_t* positions, const int32_t* seq_len, const int32_t* bt,
-                                  int64_t bt_stride, const float* sink, const void* gate, int64_t ldg, int n_tokens, int H, int G, int Gv,
+                                  int64_t bt_stride, const float* sink, const void* gate, int64_t ldg, int gate_el, int n_tokens, int H, int G, int Gv,
                                   int d, int dv, int page, int mask_kind, int mask, int keep_first, float softcap, float scale,
                                   int only_single, int out_f32) {
-#define SINK_PLAIN_ARGS st, q, kc, vc, out, tok_seq, positions, seq_len, bt, bt_stride, sink, gate, ldg, n_tokens, H, G, Gv, d, dv, page, mask_kind, mask, keep_first, softcap, scale, only_single, out_f32
+#define SINK_PLAIN_ARGS st, q, kc, vc, out, tok_seq, positions, seq_len, bt, bt_stride, sink, gate, ldg, gate_el, n_tokens, H, G, Gv, d, dv, page, mask_kind, mask, keep_first, softcap, scale, only_single, out_f32
   // heads of a group that share a CTA: as many as divide the group, up to four (two for wide values: registers)
   if (rep % 4 == 0 && dv <= 128) launch_sink_plain<T, 4>(SINK_PLAIN_ARGS);
   else if (rep % 2 == 0) launch_sink_plain<T, 2>(SINK_PLAIN_ARGS);
@@ -288,7 +289,7 @@ __global__ void __launch_bounds__(SD_WARPS * 32)
 sink_attn_decode_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache, T* __restrict__ out,
                         const int32_t* __restrict__ seq_start, const int32_t* __restrict__ seq_pos0,
                         const int32_t* __restrict__ seq_len, const int32_t* __restrict__ block_tables, int64_t bt_stride,
-                        const float* __restrict__ sink, const T* __restrict__ gate, int64_t ldg, int H, int G, int Gv, int page,
+                        const float* __restrict__ sink, const T* __restrict__ gate, int64_t ldg, int gate_el, int H, int G, int Gv, int page,
                         int mask_kind, int mask, int keep_first, float softcap, float scale, int out_f32) {
   constexpr int N = Vec16<T>::N, D = LPK * N, DV = D * VR, KPW = 32 / LPK;
   constexpr float LOG2E = 1.4426950408889634f;
@@ -433,13 +434,14 @@ sink_attn_decode_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
       den += cw[w] * part[w][r][DV + 1];
     }
     float gv = 1.f;
-    if (gate != nullptr) gv = sigmoid_f(to_f(gate[t * ldg + h]));
+    if (gate != nullptr && !gate_el) gv = sigmoid_f(to_f(gate[t * ldg + h]));
     const float inv = gv / den;
     const size_t obase = (t * H + h) * DV;
     for (int c = threadIdx.x; c < DV; c += blockDim.x) {
       float o = 0.f;
 #pragma unroll
       for (int w = 0; w < SD_WARPS; ++w) o += cw[w] * part[w][r][c];
+      if (gate != nullptr && gate_el) o *= sigmoid_f(to_f(gate[t * ldg + static_cast<int64_t>(h) * DV + c]));
       put_out(out, obase + c, o * inv, out_f32);
     }
   }
@@ -448,11 +450,11 @@ sink_attn_decode_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
 template <typename T, int LPK, int VR>
 static void launch_sink_decode(int rep, cudaStream_t st, const void* q, const void* kc, const void* vc, void* out,
                                const int32_t* seq_start, const int32_t* seq_pos0, const int32_t* seq_len, const int32_t* bt,
-                               int64_t bt_stride, const float* sink, const void* gate, int64_t ldg, int n_seqs, int H, int G, int Gv,
+                               int64_t bt_stride, const float* sink, const void* gate, int64_t ldg, int gate_el, int n_seqs, int H, int G, int Gv,
                                int page, int mask_kind, int mask, int keep_first, float softcap, float scale, int out_f32) {
 #define SD_GO(REP) sink_attn_decode_kernel<T, LPK, REP, VR><<<dim3(H / REP, n_seqs), SD_WARPS * 32, 0, st>>>(static_cast<const T*>(q), \
       static_cast<const T*>(kc), static_cast<const T*>(vc), static_cast<T*>(out), seq_start, seq_pos0, seq_len, bt, bt_stride, sink, \
-      static_cast<const T*>(gate), ldg, H, G, Gv, page, mask_kind, mask, keep_first, softcap, scale, out_f32)
+      static_cast<const T*>(gate), ldg, gate_el, H, G, Gv, page, mask_kind, mask, keep_first, softcap, scale, out_f32)
   if constexpr (LPK * Vec16<T>::N * VR <= 128) {          // four heads' accumulators fit registers and shared memory
     if (rep % 4 == 0) { SD_GO(4); return; }
   }
@@ -465,12 +467,12 @@ static void launch_sink_decode(int rep, cudaStream_t st, const void* q, const vo
 template <typename T>
 static bool launch_sink_decode_any(int d, int dv, int rep, cudaStream_t st, const void* q, const void* kc, const void* vc, void* out,
                                    const int32_t* seq_start, const int32_t* seq_pos0, const int32_t* seq_len, const int32_t* bt,
-                                   int64_t bt_stride, const float* sink, const void* gate, int64_t ldg, int n_seqs, int H, int G, int Gv,
+                                   int64_t bt_stride, const float* sink, const void* gate, int64_t ldg, int gate_el, int n_seqs, int H, int G, int Gv,
                                    int page, int mask_kind, int mask, int keep_first, float softcap, float scale, int out_f32) {
   constexpr int N = Vec16<T>::N;
   if ((dv != d && dv != 2 * d) || d % N != 0) return false;
   const bool wide = dv == 2 * d;
-#define SD_ARGS rep, st, q, kc, vc, out, seq_start, seq_pos0, seq_len, bt, bt_stride, sink, gate, ldg, n_seqs, H, G, Gv, page, mask_kind, mask, keep_first, softcap, scale, out_f32
+#define SD_ARGS rep, st, q, kc, vc, out, seq_start, seq_pos0, seq_len, bt, bt_stride, sink, gate, ldg, gate_el, n_seqs, H, G, Gv, page, mask_kind, mask, keep_first, softcap, scale, out_f32
   switch (d / N) {
     case 4: if (wide) launch_sink_decode<T, 4, 2>(SD_ARGS); else launch_sink_decode<T, 4, 1>(SD_ARGS); return true;
     case 8: if (wide) launch_sink_decode<T, 8, 2>(SD_ARGS); else launch_sink_decode<T, 8, 1>(SD_ARGS); return true;
@@ -514,7 +516,7 @@ sink_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* _
                      const __nv_bfloat16* __restrict__ v_cache, __nv_bfloat16* __restrict__ out,
                      const int32_t* __restrict__ seq_start, const int32_t* __restrict__ seq_pos0,
                      const int32_t* __restrict__ seq_len, const int32_t* __restrict__ block_tables, int64_t bt_stride,
-                     const float* __restrict__ sink, const __nv_bfloat16* __restrict__ gate, int64_t ldg, int H, int G, int Gv,
+                     const float* __restrict__ sink, const __nv_bfloat16* __restrict__ gate, int64_t ldg, int gate_el, int H, int G, int Gv,
                      int page, int mask_kind, int mask, int keep_first, float softcap, float scale, int out_f32) {
   constexpr int QS = D + 8, VS = DV + 8;             // padded rows: 16-byte aligned, ldmatrix rows land in distinct banks
   constexpr float LOG2E = 1.4426950408889634f;
@@ -677,8 +679,17 @@ sink_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* _
     if (!(half ? ok_hi : ok_lo)) continue;
     const size_t row = static_cast<size_t>(start + t0 + row_lo + 8 * half);
     float inv = 1.0f / (half ? l1 : l0);
-    if (gate != nullptr) inv *= sigmoid_f(__bfloat162float(gate[row * ldg + h]));
+    if (gate != nullptr && !gate_el) inv *= sigmoid_f(__bfloat162float(gate[row * ldg + h]));
     const size_t obase = (row * H + h) * DV + 2 * (lane & 3);
+    if (gate != nullptr && gate_el) {                // a pair of columns per load: the caller checked the alignment
+      const __nv_bfloat16* gr = gate + row * ldg + h * DV + 2 * (lane & 3);
+#pragma unroll
+      for (int nt = 0; nt < DV / 8; ++nt) {
+        const uint32_t gw = *reinterpret_cast<const uint32_t*>(gr + nt * 8);
+        oacc[nt][2 * half] *= sigmoid_f(bf16lo(gw));
+        oacc[nt][2 * half + 1] *= sigmoid_f(bf16hi(gw));
+      }
+    }
     if (out_f32) {
       float* o = reinterpret_cast<float*>(out) + obase;
 #pragma unroll
@@ -696,7 +707,7 @@ sink_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* _
 template <int D, int DV>
 static cudaError_t launch_sink_mma(int max_new, int n_seqs, cudaStream_t st, const void* q, const void* kc, const void* vc, void* out,
                                    const int32_t* seq_start, const int32_t* seq_pos0, const int32_t* seq_len, const int32_t* bt,
-                                   int64_t bt_stride, const float* sink, const void* gate, int64_t ldg, int H, int G, int Gv, int page,
+                                   int64_t bt_stride, const float* sink, const void* gate, int64_t ldg, int gate_el, int H, int G, int Gv, int page,
                                    int mask_kind, int mask, int keep_first, float softcap, float scale, int out_f32) {
   auto kern = sink_attn_mma_kernel<D, DV>;
   const size_t smem = sizeof(__nv_bfloat16) * ((SM_BM + 2 * SM_BN) * (D + 8) + 2 * SM_BN * (DV + 8));
@@ -709,7 +720,7 @@ static cudaError_t launch_sink_mma(int max_new, int n_seqs, cudaStream_t st, con
   using B = __nv_bfloat16;
   const dim3 grid((max_new + SM_BM - 1) / SM_BM, H, n_seqs);
   kern<<<grid, 128, smem, st>>>(static_cast<const B*>(q), static_cast<const B*>(kc), static_cast<const B*>(vc), static_cast<B*>(out),
-                                seq_start, seq_pos0, seq_len, bt, bt_stride, sink, static_cast<const B*>(gate), ldg, H, G, Gv, page,
+                                seq_start, seq_pos0, seq_len, bt, bt_stride, sink, static_cast<const B*>(gate), ldg, gate_el, H, G, Gv, page,
                                 mask_kind, mask, keep_first, softcap, scale, out_f32);
   return cudaSuccess;
 }
@@ -719,11 +730,11 @@ static bool sink_mma_shape(int d, int dv) {
   return (d == 32 || d == 48 || d == 64 || d == 96 || d == 128) && (dv == 64 || dv == 128);
 }
 
-#define SINK_MMA_ARGS max_new, n_seqs, st, q, kc, vc, out, seq_start, seq_pos0, seq_len, bt, bt_stride, sink, gate, ldg, H, G, Gv, page, mask_kind, mask, keep_first, softcap, scale, out_f32
+#define SINK_MMA_ARGS max_new, n_seqs, st, q, kc, vc, out, seq_start, seq_pos0, seq_len, bt, bt_stride, sink, gate, ldg, gate_el, H, G, Gv, page, mask_kind, mask, keep_first, softcap, scale, out_f32
 template <int D>
 static cudaError_t launch_sink_mma_dv(int dv, int max_new, int n_seqs, cudaStream_t st, const void* q, const void* kc, const void* vc,
                                       void* out, const int32_t* seq_start, const int32_t* seq_pos0, const int32_t* seq_len,
-                                      const int32_t* bt, int64_t bt_stride, const float* sink, const void* gate, int64_t ldg, int H,
+                                      const int32_t* bt, int64_t bt_stride, const float* sink, const void* gate, int64_t ldg, int gate_el, int H,
                                       int G, int Gv, int page, int mask_kind, int mask, int keep_first, float softcap, float scale,
                                       int out_f32) {
   return dv == 64 ? launch_sink_mma<D, 64>(SINK_MMA_ARGS) : launch_sink_mma<D, 128>(SINK_MMA_ARGS);
@@ -737,7 +748,7 @@ using namespace b2::row;
 
 extern "C" int b2tts_sink_attn(const void* q, const void* k_cache, const void* v_cache, void* out, const int32_t* tok_seq,
                                const int32_t* positions, const int32_t* seq_start, const int32_t* seq_pos0, const int32_t* seq_len,
-                               const int32_t* block_tables, int64_t bt_stride, const float* sink, const void* gate, int64_t ldg,
+                               const int32_t* block_tables, int64_t bt_stride, const float* sink, const void* gate, int64_t ldg, int gate_el,
                                int n_tokens, int n_seqs, int max_new, int heads, int kv_heads, int v_heads, int dim, int vdim, int page,
                                int mask_kind, int mask, int keep_first, float softcap, float scale, int dtype, int path, int out_f32,
                                void* stream) {
@@ -757,7 +768,8 @@ extern "C" int b2tts_sink_attn(const void* q, const void* k_cache, const void* v
              "sink_attn: null pointer");
   B2_REQUIRE(aligned16(k_cache) && aligned16(v_cache), B2TTS_EALIGN, "sink_attn: caches must be 16-byte aligned");
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const bool mma_ok = dtype == B2TTS_DTYPE_BF16 && sink_mma_shape(dim, vdim) && aligned16(q) && aligned16(out);
+  const bool mma_ok = dtype == B2TTS_DTYPE_BF16 && sink_mma_shape(dim, vdim) && aligned16(q) && aligned16(out) &&
+                      (!gate || !gate_el || (reinterpret_cast<uintptr_t>(gate) % 4 == 0 && ldg % 2 == 0));
   B2_REQUIRE(path != 2 || mma_ok, B2TTS_EUNSUPPORTED, "sink_attn: the tensor-core kernel takes bf16 with head sizes 32..128 / 64, 128");
   const bool use_mma = mma_ok && path != 1 && max_new > 1;
   if (use_mma) {
@@ -779,11 +791,11 @@ extern "C" int b2tts_sink_attn(const void* q, const void* k_cache, const void* v
   if (path != 1 && aligned16(q) && n_seqs > 0) {
     if (dtype == B2TTS_DTYPE_BF16)
       split = launch_sink_decode_any<__nv_bfloat16>(dim, vdim, heads / kv_heads, st, q, k_cache, v_cache, out, seq_start, seq_pos0, seq_len,
-                                                    block_tables, bt_stride, sink, gate, ldg, n_seqs, heads, kv_heads, v_heads, page, mask_kind,
+                                                    block_tables, bt_stride, sink, gate, ldg, gate_el, n_seqs, heads, kv_heads, v_heads, page, mask_kind,
                                                     mask, keep_first, softcap, scale, out_f32);
     else
       split = launch_sink_decode_any<float>(dim, vdim, heads / kv_heads, st, q, k_cache, v_cache, out, seq_start, seq_pos0, seq_len,
-                                            block_tables, bt_stride, sink, gate, ldg, n_seqs, heads, kv_heads, v_heads, page, mask_kind, mask,
+                                            block_tables, bt_stride, sink, gate, ldg, gate_el, n_seqs, heads, kv_heads, v_heads, page, mask_kind, mask,
                                             keep_first, softcap, scale, out_f32);
     if (split) B2_CHECK_LAUNCH("sink_attn (one-token rows)");
   }
@@ -791,11 +803,11 @@ extern "C" int b2tts_sink_attn(const void* q, const void* k_cache, const void* v
   const int skip = (use_mma ? 1 : 0) | (split ? 2 : 0);
   if (dtype == B2TTS_DTYPE_BF16)
     launch_sink_plain_rep<__nv_bfloat16>(heads / kv_heads, st, q, k_cache, v_cache, out, tok_seq, positions, seq_len, block_tables,
-                                         bt_stride, sink, gate, ldg, n_tokens, heads, kv_heads, v_heads, dim, vdim, page, mask_kind, mask,
+                                         bt_stride, sink, gate, ldg, gate_el, n_tokens, heads, kv_heads, v_heads, dim, vdim, page, mask_kind, mask,
                                          keep_first, softcap, scale, skip, out_f32);
   else
     launch_sink_plain_rep<float>(heads / kv_heads, st, q, k_cache, v_cache, out, tok_seq, positions, seq_len, block_tables, bt_stride,
-                                 sink, gate, ldg, n_tokens, heads, kv_heads, v_heads, dim, vdim, page, mask_kind, mask, keep_first,
+                                 sink, gate, ldg, gate_el, n_tokens, heads, kv_heads, v_heads, dim, vdim, page, mask_kind, mask, keep_first,
                                  softcap, scale, skip, out_f32);
   B2_CHECK_LAUNCH("sink_attn");
   return B2TTS_OK;

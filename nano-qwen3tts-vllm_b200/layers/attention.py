@@ -118,17 +118,22 @@ class SinkSoftmaxAttention(nn.Module):
     into c tanh(s / c); ``keep_first`` keys stay visible behind the mask; ``mask`` 0 is plain causal attention; the
     rotation pairs coordinate i with i + dims/2 or 2i with 2i + 1 as the ``rotary`` module says; ``v_heads`` < ``kv_heads``
     value heads are shared by the key heads (key head g reads value head g mod v_heads); ``own_cache`` False: the
-    module projects no keys and values and reads a cache another module writes."""
+    module projects no keys and values and reads a cache another module writes; ``head_norm``: RMS norm of every q and k
+    HEAD with one weight of ``dim`` for q and one for k, in front of the rotation (which then comes from the step's table:
+    ``rotary`` is a ``PairRotaryTable`` or ``HalfRotaryTable``); ``element_gate``: the gate has one number per output element."""
 
     MASKS = {"window": nat.MASK_WINDOW, "chunk": nat.MASK_CHUNK}
 
     def __init__(self, heads: int, kv_heads: int, dim: int, vdim: int, mask_kind: str, mask: int, scale: float, *,
                  bias: bool = False, qk_norm: bool = False, rotary=None, eps: float = 1e-6, sink: str = "learned",
-                 softcap: float = 0.0, keep_first: int = 0, v_heads: int | None = None, own_cache: bool = True):
+                 softcap: float = 0.0, keep_first: int = 0, v_heads: int | None = None, own_cache: bool = True,
+                 head_norm: bool = False, element_gate: bool = False):
         super().__init__()
+        assert not (head_norm and (qk_norm or (v_heads or kv_heads) != kv_heads or not own_cache))
         assert sink in ("learned", "zero", "none")
         self.heads, self.kv_heads, self.dim, self.vdim, self.scale, self.eps = heads, kv_heads, dim, vdim, scale, eps
         self.mask_kind, self.mask, self.rotary = self.MASKS[mask_kind], mask, rotary
+        self.head_norm, self.element_gate = head_norm, element_gate
         self.softcap, self.keep_first, self.v_heads, self.own_cache = softcap, keep_first, v_heads or kv_heads, own_cache
         f32 = dict(dtype=torch.float32)
         self.sink = nn.Parameter(torch.zeros(heads, **f32), requires_grad=False) if sink != "none" else None
@@ -136,8 +141,8 @@ class SinkSoftmaxAttention(nn.Module):
         self.q_bias = mk(heads * dim, False) if bias else None
         self.k_bias = mk(kv_heads * dim, False) if bias else None
         self.v_bias = mk(kv_heads * vdim, False) if bias else None
-        self.q_norm = mk(heads * dim, True) if qk_norm else None
-        self.k_norm = mk(kv_heads * dim, True) if qk_norm else None
+        self.q_norm = mk(dim if head_norm else heads * dim, True) if qk_norm or head_norm else None
+        self.k_norm = mk(dim if head_norm else kv_heads * dim, True) if qk_norm or head_norm else None
         self.k_cache = self.v_cache = torch.tensor([])
 
     def prepare(self, u: torch.Tensor, q_off: int, k_off: int, v_off: int) -> torch.Tensor:
@@ -145,6 +150,11 @@ class SinkSoftmaxAttention(nn.Module):
         q = torch.empty(u.shape[0], self.heads * self.dim, dtype=u.dtype, device=u.device)
         rot = self.rotary
         own = self.own_cache
+        if self.head_norm:
+            nat.attn_head_prep(u, q_off, k_off, v_off, self.q_bias, self.k_bias, self.v_bias, self.q_norm, self.k_norm,
+                               rot.table if rot is not None else None, rot is not None and rot.interleaved, lay, q, self.k_cache,
+                               self.v_cache, self.heads, self.kv_heads, self.dim, self.vdim, self.eps)
+            return q
         nat.attn_prep(u, q_off, k_off, v_off, self.q_bias, self.k_bias, self.v_bias if v_off >= 0 else None, self.q_norm,
                       self.k_norm, rot.freq if rot is not None else None, rot.dims if rot is not None else 0, lay, q,
                       self.k_cache if own else None, self.v_cache if own else None, self.heads, self.kv_heads, self.dim,
@@ -157,7 +167,7 @@ class SinkSoftmaxAttention(nn.Module):
         out = torch.empty(q.shape[0], self.heads * self.vdim, dtype=out_dtype or q.dtype, device=q.device)
         nat.sink_attn(q, self.k_cache, self.v_cache, out, lay, self.sink, gate, self.heads, self.kv_heads, self.dim, self.vdim,
                       self.k_cache.shape[1], self.mask_kind, self.mask, self.scale, v_heads=self.v_heads,
-                      keep_first=self.keep_first, softcap=self.softcap)
+                      keep_first=self.keep_first, softcap=self.softcap, gate_el=self.element_gate)
         return out
 
 

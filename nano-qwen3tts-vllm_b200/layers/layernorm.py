@@ -118,6 +118,42 @@ class OffsetRMSNorm(nn.Module):
         return nat.gather_group_norm(x, rows, self.weight, 1, self.eps, dtype)
 
 
+class DynamicTanh(nn.Module):
+    """A norm without statistics: D(v) = tanh(alpha v) * w + b with one number ``alpha`` and two vectors, all kept in float.  In
+    a model it rides in the residual update in front of it (``TanhSandwich``); ``forward`` is the stand-alone form over a
+    subset of rows (the final norm)."""
+
+    def __init__(self, width: int):
+        super().__init__()
+        f32 = dict(dtype=torch.float32)
+        self.weight = nn.Parameter(torch.ones(width, **f32), requires_grad=False)
+        self.bias = nn.Parameter(torch.zeros(width, **f32), requires_grad=False)
+        self.alpha = nn.Parameter(torch.ones((), **f32), requires_grad=False)
+
+    def args(self) -> tuple:
+        return self.weight, self.bias, self.alpha.view(1)
+
+    def forward(self, x: torch.Tensor, dtype: torch.dtype, rows: torch.Tensor | None = None) -> torch.Tensor:
+        return nat.tanh_gather(x, rows, self.args(), dtype)
+
+
+class TanhSandwich(nn.Module):
+    """The pair of dynamic tanhs around a sublayer: ``self.pre`` on the way in, ``self.post`` on the way out, the result times
+    ``mult``.  ``add`` does x += mult * post(y) on a 32-bit stream and, in the same launch, makes what comes next: ``nxt(x)`` (a
+    ``DynamicTanh``), or the operand of a pass's input projection (``layers/pass_input.py``).  y is a dense output ``a``, the weighted
+    expert outputs ``z`` / ``zw`` of a mixture, or both."""
+
+    def __init__(self, width: int, mult: float):
+        super().__init__()
+        self.mult, self.pre, self.post = mult, DynamicTanh(width), DynamicTanh(width)
+
+    def add(self, x: torch.Tensor, nxt: "DynamicTanh | None", *, a=None, z=None, zw=None, cat_with: tuple | None = None) -> torch.Tensor | None:
+        """``cat_with`` = (table, row indices): return the stream beside those rows instead of ``nxt(x)``."""
+        kw = dict(table=cat_with[0], index=cat_with[1], want_cat=True) if cat_with is not None else \
+            dict(pre=nxt.args() if nxt is not None else None)
+        return nat.tanh_residual(x, a=a, z=z, zw=zw, post=self.post.args(), mult=self.mult, **kw)
+
+
 class GatedResidual(nn.Module):
     """Gate of a sublayer's result on its way into a 32-bit residual stream: x += sigmoid(z + b) * y with z = W h, h the
     sublayer's input (W rides in a projection of the sublayer; the bias is kept here in float).  ``forward`` updates x in

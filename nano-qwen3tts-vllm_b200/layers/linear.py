@@ -168,6 +168,33 @@ def linear_gelu_mul(x: torch.Tensor, gate_up_weight: torch.Tensor) -> torch.Tens
     return nat.gelu_mul(linear(x, gate_up_weight))
 
 
+def linear_clamped_gate(x: torch.Tensor, gate_up_weight: torch.Tensor, limit: float, alpha: float = nat.GATE_SIGMOID_SCALE) -> torch.Tensor:
+    """g sigmoid(alpha g) (u + 1), g = min(x Wg^T, limit), u = clamp(x Wu^T, -limit, limit), over the merged [gate; up] weight, with
+    the activation in the GEMM epilogue on the native path; the library GEMM followed by the gated product elsewhere (long
+    prompts, float32)."""
+    m, n = x.shape[0], gate_up_weight.shape[0]
+    if x.dtype == torch.bfloat16 and native_ok(m, n, x.shape[1]):
+        return nat.gemm_clamped_gate(x, packed_weight(gate_up_weight, nat.PACK_GATE_UP), n, limit, alpha, pdl=PDL)
+    return nat.clamped_gate_mul(linear(x, gate_up_weight), limit, alpha)
+
+
+def linear_float(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
+    """x W^T (+ b) as FLOATS: bfloat16 operands whose float sums leave the GEMM unrounded (the native kernel, or the library's
+    with a float output).  ``bias`` has x's dtype."""
+    m, n = x.shape[0], weight.shape[0]
+    if out is None:
+        out = torch.empty(m, n, dtype=torch.float32, device=x.device)
+    if m == 0:
+        return out
+    if x.dtype == torch.bfloat16 and native_ok(m, n, x.shape[1]):
+        return nat.gemm_f32out(x, packed_weight(weight), n, bias=bias, out=out, pdl=PDL)
+    if x.dtype == torch.bfloat16:
+        torch.mm(x, weight.t(), out_dtype=torch.float32, out=out)
+    else:
+        torch.mm(x, weight.t(), out=out)
+    return out.add_(bias) if bias is not None else out
+
+
 def per_head_linear(x: torch.Tensor, weight: torch.Tensor, transpose_weight: bool = False) -> torch.Tensor:
     """One small projection per head, all heads in one strided-batched library GEMM (cuBLAS through ``torch.bmm``):
     x [heads, n, k] (any strides) and weight [heads, k, m] (or [heads, m, k] with ``transpose_weight``) -> [heads, n, m]."""

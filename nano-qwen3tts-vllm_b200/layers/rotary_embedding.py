@@ -100,6 +100,19 @@ class PairRotary(nn.Module):
     interleaved = True
 
 
+class PairRotaryTable(PairRotary):
+    """The same rotation for kernels that read cosines and sines from a table: ``fill`` computes the table of a step's
+    positions once ([n, dims]: cosines, then sines), every layer with the same frequencies then shares ``table``."""
+
+    def __init__(self, dims: int, base: float, scaling: dict | None = None):
+        super().__init__(dims, base, scaling)
+        assert self.mult == 1.0                # the table holds plain cosines and sines
+        self.table = None
+
+    def fill(self, positions: torch.Tensor) -> None:
+        self.table = nat.rotary_table(positions, self.freq)
+
+
 class HalfRotary(nn.Module):
     """Frequencies of a rotation that pairs coordinate i with i + dims/2 (i < dims/2) of the first ``dims`` coordinates
     of a head: f_i = base^(-2i/dims).  Computed in float64, kept as float; the kernel that rotates

@@ -64,6 +64,9 @@ register(Architecture("Zekivik", ".config:ZekivikConfig", ".models.zekivik:Zekiv
 register(Architecture("Teberax", ".config:TeberaxConfig", ".models.teberax:TeberaxForCausalLM",
                       ".engine.model_runner.lm_model_runner:LMModelRunner",
                       ".engine.llm_engine.lm_engine:CausalLMEngine"))
+register(Architecture("Gekavik", ".config:GekavikConfig", ".models.gekavik:GekavikForCausalLM",
+                      ".engine.model_runner.lm_model_runner:LMModelRunner",
+                      ".engine.llm_engine.lm_engine:CausalLMEngine"))
 
 
 def resolve(config: dict) -> Architecture:

@@ -44,8 +44,9 @@ class LatentAttentionMixer(nn.Module):
         self.eps = eps
         self.q_size = m.heads * (m.dim + m.rot_dim)
         self.q_in = m.q_rank if m.q_rank else self.q_size
-        parts = [self.q_in, m.kv_rank + m.rot_dim] + ([m.heads * m.vdim] if m.gate else [])
-        self.in_proj = MergedColumnParallelLinear(width, parts)                 # [dq | q ; dkv ; g]
+        # the last part is a gate per output element, or per head: an odd width, padded to whole tiles of the native GEMM
+        parts = [self.q_in, m.kv_rank + m.rot_dim] + ([m.heads * (1 if m.head_gate else m.vdim)] if m.gate else [])
+        self.in_proj = MergedColumnParallelLinear(width, parts, pad_to=128 if m.head_gate else 1)       # [dq | q ; dkv ; g]
         f32 = dict(dtype=torch.float32)
         if m.q_rank:
             self.q_norm = nn.Parameter(torch.ones(m.q_rank, **f32), requires_grad=False)
@@ -77,7 +78,7 @@ class LatentAttentionMixer(nn.Module):
         v = per_head_linear(o, self.uv, transpose_weight=True)                   # [heads, n, vdim]
         heads_out = torch.empty(n, m.heads * m.vdim, dtype=hs.dtype, device=hs.device)
         gate = u[:, self.q_in + m.kv_rank + m.rot_dim:] if m.gate else None
-        nat.gate_heads(v, (m.vdim, n * m.vdim), gate, heads_out, m.heads, m.vdim)
+        nat.gate_heads(v, (m.vdim, n * m.vdim), gate, heads_out, m.heads, m.vdim, per_head=m.head_gate)
         return self.o_proj(heads_out)
 
 

@@ -36,6 +36,7 @@ from ..layers.linear import ColumnParallelLinear, MergedColumnParallelLinear, Ro
 from ..layers.moe import SoftmaxIdentityMoE
 from ..layers.recurrent import GatedLinearAttention
 from ..layers.rotary_embedding import PairRotary
+from .checkpoint import load_targets
 from .ridevik import LatentAttentionMixer
 
 F32 = dict(dtype=torch.float32)
@@ -293,30 +294,10 @@ class TeberaxForCausalLM(nn.Module):
         the mixer's tensors under ``l<i>.mix.`` (a parallel mixer's under ``.left.`` / ``.right.``) and the feed-forward's
         under ``l<i>.mlp.`` (experts ``.e<j>.``).  Tensors are bfloat16 in the file; what the kernels keep in float (norm
         gains and weights, biases of the attention, routers, the numbers of activations and of lambda) is widened exactly."""
-        targets, seen = self._targets(), set()
-        for name, value in state_dict.items():
-            if name not in targets:
-                if strict:
-                    raise KeyError(f"unexpected tensor {name!r} in the checkpoint")
-                continue
-            param, shard, transform = targets[name]
-            if transform is not None:
-                value = transform(value)
-            with torch.no_grad():
-                if shard is not None:
-                    param.weight_loader(param, value.to(param.dtype), shard)
-                else:
-                    if param.numel() != value.numel() or (param.dim() == value.dim() and tuple(param.shape) != tuple(value.shape)):
-                        raise ValueError(f"{name}: shape {tuple(value.shape)} does not fit {tuple(param.shape)}")
-                    param.copy_(value.to(param.dtype).reshape(param.shape))
-            seen.add(name)
+        seen = load_targets(self._targets(), state_dict, strict)
         for layer in self.layers:
             if layer.kind == "attention":
                 layer.mix.attn._lam = None
-        if strict:
-            missing = sorted(set(targets) - seen)
-            if missing:
-                raise KeyError(f"missing tensors: {missing[:8]}{' ...' if len(missing) > 8 else ''}")
         return seen
 
 

@@ -31,6 +31,7 @@ from ..layers.linear import ColumnParallelLinear, MergedColumnParallelLinear, Ro
 from ..layers.recurrent import Retention
 from ..layers.rotary_embedding import HalfRotaryTable
 from ..layers.short_conv import ShortConvRotaryQKV
+from .checkpoint import load_targets
 
 GEMM_ROWS = 128          # the native GEMM's output tile: merged input projections are padded to whole tiles
 
@@ -232,28 +233,7 @@ class ZekivikForCausalLM(nn.Module):
         ``l<i>.rg1|rg2`` with ``.b``, the mixer's tensors under ``l<i>.mix.`` and the feed-forward's under ``l<i>.mlp.``.
         Tensors are bfloat16 in the file; what the kernels keep in float (norm weights plus one, gate biases, filters, the
         passes' vectors) is widened exactly."""
-        targets, seen = self._targets(), set()
-        for name, value in state_dict.items():
-            if name not in targets:
-                if strict:
-                    raise KeyError(f"unexpected tensor {name!r} in the checkpoint")
-                continue
-            param, shard, transform = targets[name]
-            if transform is not None:
-                value = transform(value)
-            with torch.no_grad():
-                if shard is not None:
-                    param.weight_loader(param, value.to(param.dtype), shard)
-                else:
-                    if tuple(param.shape) != tuple(value.shape):
-                        raise ValueError(f"{name}: shape {tuple(value.shape)} does not fit {tuple(param.shape)}")
-                    param.copy_(value.to(param.dtype))
-            seen.add(name)
-        if strict:
-            missing = sorted(set(targets) - seen)
-            if missing:
-                raise KeyError(f"missing tensors: {missing[:8]}{' ...' if len(missing) > 8 else ''}")
-        return seen
+        return load_targets(self._targets(), state_dict, strict)
 
 
 def checkpoint_shapes(config: ZekivikConfig) -> dict:
