@@ -170,7 +170,7 @@ def random_config(vocab=61, width=24, types=("attention", "latent_attention", "a
     att.update(attention or {})
     lat = dict(heads=3, dim=6, vdim=5, kv_rank=12, q_rank=7, scale=0.35, mask={"size": 11})
     lat.update(latent or {})
-    me = dict(kind="moe", expert={"ff": 10, "limit": 0.8}, router={"experts": 6, "top": 2, "groups": {"count": 3, "keep": 2}},
+    me = dict(kind="moe", expert={"ff": 10, "limit": 0.8}, router={"experts": 8, "top": 3, "groups": {"count": 4, "keep": 2}},
               shared={"ff": 9, "limit": 1.5})
     me.update(moe or {})
     layers = [{"type": kind, "mixer": dict(att if kind == "attention" else lat), "mlp": None if ff[i % len(ff)] is None else dict(me)}
