@@ -71,6 +71,10 @@ def parse():
                     help="instead of the frame loop: the Zekivik decoder (convolved unit-norm attention, fixed-decay retention, gated "
                          "residuals) beside Teberax at equal layer sizes, plus the kernels of both against their rooflines "
                          "(bench_lm.py); one JSON line")
+    ap.add_argument("--lm-gekavik", action="store_true",
+                    help="instead of the frame loop: the Gekavik decoder (dynamic-tanh norms, gated window attention, latent attention, "
+                         "group-limited clamped experts, looped layers) beside Teberax and Ridevik at equal layer sizes, plus the kernels "
+                         "of all three against their rooflines (bench_lm.py); one JSON line")
     return ap.parse_args()
 
 
@@ -494,11 +498,11 @@ def main():
         dist.init_process_group("nccl", device_id=torch.device(device))
     barrier = (lambda: (dist.barrier(), torch.cuda.synchronize())) if dist else None
 
-    if a.lm or a.lm_latent or a.lm_hybrid or a.lm_teberax or a.lm_zekivik:
+    lm = next((name for name in ("gekavik", "zekivik", "teberax", "hybrid", "latent") if getattr(a, "lm_" + name)), None)
+    if a.lm or lm:
         import bench_lm
         if rank == 0:
-            run = bench_lm.main_zekivik if a.lm_zekivik else bench_lm.main_teberax if a.lm_teberax else bench_lm.main_hybrid if a.lm_hybrid else bench_lm.main_latent if a.lm_latent \
-                else bench_lm.main
+            run = getattr(bench_lm, "main_" + lm) if lm else bench_lm.main
             print(json.dumps(run(device)), flush=True)
         return
 

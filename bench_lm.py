@@ -69,7 +69,7 @@ def bench_bokenex(s: dict, moe: bool, device: str, design: str = "bokenex") -> d
     from nano_qwen3tts_vllm_b200.engine.llm_engine.lm_engine import CausalLMEngine
     from nano_qwen3tts_vllm_b200.sampling_params import SamplingParams
     cfg = {"bokenex": bokenex_config, "ridevik": ridevik_config, "tibivik": tibivik_config, "teberax": teberax_config,
-           "zekivik": zekivik_config}[design](s, moe)
+           "zekivik": zekivik_config, "gekavik": gekavik_config, "gekavik_looped": gekavik_looped_config}[design](s, moe)
     pages = DECODE_SEQS * ((DECODE_CTX + 64 + PAGE - 1) // PAGE) + PREFILL_SEQS * (PREFILL_LEN // PAGE + 1)
     eng = CausalLMEngine(cfg, state_dict="random:7", kvcache_block_size=PAGE, num_kvcache_blocks=pages,
                          max_num_seqs=DECODE_SEQS + PREFILL_SEQS, max_model_len=4096, max_num_batched_tokens=16384,
@@ -899,6 +899,187 @@ def main_zekivik(device: str = "cuda:0") -> dict:
     out["like_kernels"] = {**bench_teberax_kernels(device),
                            **{k: v for k, v in bench_kernels(device).items() if k.startswith("conv_headnorm")},
                            **{k: v for k, v in bench_hybrid_kernels(device).items() if k.startswith(("gated_group_norm", "sink_attn"))}}
+    out["seconds"] = round(time.time() - t0, 1)
+    return out
+
+
+def gekavik_config(s: dict, moe: bool = True, loop: dict | None = None):
+    """Layers of real models' shapes at the size's width: three window attentions of the size's head layout with four kept
+    first keys, rotated over the whole head, and one windowed latent attention over a latent of 4 head sizes; 16 clamped gated
+    experts of Teberax's inner size, top 2 out of one group of four, and a shared one of the same size."""
+    from nano_qwen3tts_vllm_b200.config import GekavikConfig
+    d, H, G, W = s["dim"], s["heads"], s["kv_heads"], s["width"]
+    ff = s["inter"] // 2
+    experts = {"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "shared": {"ff": ff, "limit": 7.0},
+               "router": {"experts": 16, "top": 2, "groups": {"count": 4, "keep": 1}}}
+    att = {"type": "attention", "mlp": experts,
+           "mixer": {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": WINDOW, "keep_first": 4},
+                     "rot": {"dims": d, "base": 1e6}}}
+    lat = {"type": "latent_attention", "mlp": experts,
+           "mixer": {"heads": H, "dim": d, "vdim": d, "kv_rank": 4 * d, "q_rank": W // 2, "scale": d ** -0.5, "mask": {"size": WINDOW}}}
+    c = {"architecture": "Gekavik", "vocab": 3072, "width": W, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "layers": [att, att, lat, att][:LAYERS]}
+    return GekavikConfig.from_dict(dict(c, loop=loop) if loop else c)
+
+
+def gekavik_looped_config(s: dict, moe: bool = True):
+    """The same layers with the first two run twice."""
+    return gekavik_config(s, moe, {"start": 0, "stop": 2, "times": 2})
+
+
+class KernelTimer:
+    """What the kernel sections share: flushed timing, step layouts, roofline entries."""
+
+    def __init__(self, device: str):
+        import torch
+        self.dev = torch.device(device)
+        self.hbm, self.tflops, self.source = _peaks()
+        self.flush = torch.empty(256 << 20, dtype=torch.uint8, device=self.dev)
+
+    def ms(self, fn, iters=7):
+        import torch
+        for _ in range(3):
+            fn()
+        ts = []
+        for _ in range(iters):
+            self.flush.zero_()
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            fn()
+            b.record()
+            torch.cuda.synchronize()
+            ts.append(a.elapsed_time(b))
+        return sorted(ts)[len(ts) // 2]
+
+    def entry(self, fn, bytes_=None, flops=None, iters=7):
+        ms = self.ms(fn, iters)
+        e = {"us": round(ms * 1e3, 1)}
+        if bytes_ is not None:
+            e["gbs"], e["frac_hbm"] = round(bytes_ / ms / 1e6, 1), round(bytes_ / ms / 1e6 / self.hbm, 3)
+        if flops is not None:
+            e["tflops"], e["frac_tensor"] = round(flops / ms / 1e9, 1), round(flops / ms / 1e9 / self.tflops, 4)
+        return e
+
+    def layout(self, n_seqs, cached, new, pages_per_seq):
+        import torch
+        from types import SimpleNamespace
+        i32 = dict(dtype=torch.int32, device=self.dev)
+        pos = (torch.arange(new, **i32) + cached).repeat(n_seqs)
+        tok_seq = torch.arange(n_seqs, **i32).repeat_interleave(new)
+        return SimpleNamespace(
+            n_seqs=n_seqs, max_new=new, n_tokens=n_seqs * new, seq_start=torch.arange(n_seqs, **i32) * new,
+            seq_pos0=torch.full((n_seqs,), cached, **i32), seq_len=torch.full((n_seqs,), new, **i32), seq_slot=torch.arange(n_seqs, **i32),
+            block_tables=torch.arange(n_seqs * pages_per_seq, **i32).view(n_seqs, pages_per_seq).contiguous(), positions=pos, tok_seq=tok_seq,
+            slot_mapping=(tok_seq * pages_per_seq * PAGE + pos).to(torch.int32))
+
+
+def bench_gekavik_kernels(device: str) -> dict:
+    """The kernels Gekavik added or extended at the w2048 layer shapes, each after an L2 flush, with the fraction of the
+    measured roofline; beside the experts' products the like launches of the SiLU-gated mixtures ("like: ...")."""
+    import torch
+    import nano_qwen3tts_vllm_b200._native as nat
+    from nano_qwen3tts_vllm_b200.layers.linear import linear_clamped_gate, linear_float, linear_silu_mul
+    from nano_qwen3tts_vllm_b200.layers.moe import SharedClampedMoE, SoftmaxIdentityMoE
+    from nano_qwen3tts_vllm_b200.layers.rotary_embedding import PairRotaryTable
+    T, BF = KernelTimer(device), torch.bfloat16
+    dev, H, G, d, D, r = T.dev, 16, 8, 128, 2048, 512
+    rnd = lambda *shape: torch.randn(*shape, device=dev).to(BF)
+    res = {"peaks": {"hbm_gbs": T.hbm, "bf16_tflops": T.tflops, "source": T.source}}
+    pps = (DECODE_CTX + PAGE) // PAGE + 1
+    steps = {f"decode {DECODE_SEQS}": T.layout(DECODE_SEQS, DECODE_CTX, 1, pps),
+             f"prefill {PREFILL_SEQS}x{PREFILL_LEN}": T.layout(PREFILL_SEQS, 0, PREFILL_LEN, PREFILL_LEN // PAGE)}
+    kc, vc, lc = (rnd(DECODE_SEQS * pps, PAGE, w) for w in (G * d, G * d, r))
+    seen = PREFILL_SEQS * sum(min(i + 1, WINDOW) for i in range(PREFILL_LEN))
+    kept = PREFILL_SEQS * sum(min(4, max(0, i + 1 - WINDOW)) for i in range(PREFILL_LEN))
+    rot = PairRotaryTable(d, 1e6).to(dev)
+    bias, nw = torch.zeros(H * d, device=dev), torch.ones(d, device=dev)
+    norm = (torch.ones(D, device=dev), torch.zeros(D, device=dev), torch.ones(1, device=dev))
+    for name, lay in steps.items():
+        n, decode = lay.n_tokens, lay.max_new == 1
+        rot.fill(lay.positions)
+        # ---- attention: preparation, window with kept keys and the element-wise gate
+        u = rnd(n, 2 * H * d + 2 * G * d)
+        q, out = torch.empty(n, H * d, dtype=BF, device=dev), torch.empty(n, H * d, dtype=BF, device=dev)
+        res[f"attn_head_prep {name}"] = T.entry(lambda: nat.attn_head_prep(
+            u, 0, H * d, (H + G) * d, bias, bias, bias, nw, nw, rot.table, True, lay, q, kc, vc, H, G, d, d, 1e-6), bytes_=n * (H + 2 * G) * d * 2 * 2)
+        gate = u[:, (H + 2 * G) * d:]
+        attn = lambda: nat.sink_attn(q, kc, vc, out, lay, None, gate, H, G, d, d, PAGE, nat.MASK_WINDOW, WINDOW, d ** -0.5, keep_first=4, gate_el=True)
+        res[f"sink_attn {name} window {WINDOW} + 4 kept, element gate"] = T.entry(
+            attn, **(dict(bytes_=n * (WINDOW + 4) * 2 * G * d * 2) if decode else dict(flops=(seen + kept) * H * 2 * d * 2)))
+        # ---- latent attention without a rotated part
+        ql = rnd(H, n, r)
+        lo = torch.empty_like(ql)
+        res[f"latent_attn {name} window {WINDOW}, no rotated part"] = T.entry(
+            lambda: nat.latent_attn(ql, (r, n * r), ql, (0, 0), lc, lo, (r, n * r), None, None, 1.0, 0, lay, H, r, 0, PAGE, WINDOW, d ** -0.5),
+            **(dict(bytes_=n * WINDOW * r * 2) if decode else dict(flops=seen * H * 2 * r * 2)))
+        v, head_gate = rnd(H, n, d), rnd(n, 128)
+        res[f"gate_heads {name}, one gate per head"] = T.entry(lambda: nat.gate_heads(v, (d, n * d), head_gate, out, H, d, per_head=True),
+                                                              bytes_=n * H * d * 2 * 2)
+        # ---- dynamic tanh, residual, next norm
+        x, a, z, zw = torch.randn(n, D, device=dev), rnd(n, D), rnd(2 * n, D), torch.rand(n, 2, device=dev)
+        res[f"tanh_residual {name} dense"] = T.entry(lambda: nat.tanh_residual(x, a=a, post=norm, mult=0.5, pre=norm), bytes_=n * D * (8 + 2 + 2))
+        res[f"tanh_residual {name} two experts + shared"] = T.entry(
+            lambda: nat.tanh_residual(x, a=a, z=z, zw=zw, post=norm, mult=0.5, pre=norm), bytes_=n * D * (8 + 3 * 2 + 2))
+        # ---- the projection in front of a pass
+        tab, ids, w3, step = rnd(3072, D), torch.randint(0, 3072, (n,), device=dev, dtype=torch.int32), rnd(D, 3 * D), rnd(D)
+        res[f"tanh_residual {name} dense, operand of a pass"] = T.entry(
+            lambda: nat.tanh_residual(x, table=tab, index=ids, a=a, post=norm, mult=0.5, want_cat=True), bytes_=n * D * (8 + 2 + 2 + 6))
+        cat = rnd(n, 3 * D)
+        res[f"pass projection {name}"] = T.entry(lambda: linear_float(cat, w3, step, out=x), bytes_=3 * D * D * 2 + n * D * (6 + 4),
+                                                flops=n * 3 * D * D * 2)
+        # ---- experts: routing, grouped products, the shared one; the SiLU-gated mixture of the same size beside them
+        prev = torch.get_default_dtype()
+        torch.set_default_dtype(BF)
+        with torch.device(dev):
+            moe, like = SharedClampedMoE(D, 3072, 16, 2, 7.0, 4, 1, 3072, 7.0), SoftmaxIdentityMoE(D, 3072, 16, 2, 0)
+        torch.set_default_dtype(prev)
+        for p in [*moe.parameters(), *like.parameters()]:
+            p.data.normal_(std=0.02)
+        h = rnd(n, D)
+        hit = min(16, 2 * n)
+        wup, wdown = hit * 2 * 3072 * D * 2, hit * 3072 * D * 2
+        ti, tw, off, sp = moe.route(h)
+        res[f"moe_route {name}, 16 experts in groups"] = T.entry(lambda: moe.route(h), bytes_=n * D * 2)
+        res[f"like: moe_route {name}, 16 experts"] = T.entry(lambda: like.route(h), bytes_=n * D * 2)
+        y = torch.empty(2 * n, 3072, dtype=BF, device=dev)
+        gu = torch.empty(2 * n, 6144, dtype=BF, device=dev)
+        cost = dict(bytes_=wup + n * D * 2 + 2 * n * 3072 * 2, flops=2 * n * 6144 * D * 2)
+
+        def unfused():
+            nat.grouped_gemm(h, like.up, gu, off, sp, 2 * n, 2, in_by_token=True, out_by_pair=False, act=0)
+            nat.silu_mul(gu)
+
+        res[f"grouped gate/up with the clamped product {name}"] = T.entry(lambda: nat.grouped_gemm_gated(h, moe.up, y, off, sp, 2 * n, 2, 7.0), **cost)
+        res[f"like: grouped gate/up, then silu_mul {name}"] = T.entry(unfused, **cost)
+        res[f"clamped_gate_mul {name}"] = T.entry(lambda: nat.clamped_gate_mul(gu, 7.0), bytes_=2 * n * 3072 * 3 * 2)
+        res[f"like: silu_mul {name}"] = T.entry(lambda: nat.silu_mul(gu), bytes_=2 * n * 3072 * 3 * 2)
+        dense = dict(bytes_=6144 * D * 2 + n * (D + 3072) * 2, flops=n * 6144 * D * 2)
+        res[f"shared expert gate/up {name}"] = T.entry(lambda: linear_clamped_gate(h, moe.shared.gate_up.weight, 7.0), **dense)
+        res[f"like: dense SiLU gate/up {name}"] = T.entry(lambda: linear_silu_mul(h, moe.shared.gate_up.weight), **dense)
+        from nano_qwen3tts_vllm_b200.layers.linear import release_packed
+        release_packed(moe)
+        del moe, like
+    return res
+
+
+def main_gekavik(device: str = "cuda:0") -> dict:
+    """``bench.py --lm-gekavik``: Gekavik (plain, and with two of its layers looped) beside Teberax (in-and-out norms, window
+    attention with kept keys, latent attention, a softmax-routed mixture) and Ridevik (latent attention and a mixture in every
+    layer) at equal width, head layout, layer count and expert sizes, then its kernels and the like kernels of both against
+    their rooflines."""
+    import torch
+    t0 = time.time()
+    out = {"metric": "lm_prefill_decode_throughput", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic (random weights)",
+           "config": {"prefill": f"{PREFILL_SEQS}x{PREFILL_LEN} tokens per step", "decode": f"{DECODE_SEQS} sequences at context {DECODE_CTX}",
+                      "layers": LAYERS, "window": WINDOW, "page": PAGE}, "sizes": {}}
+    for name, s in SIZES.items():
+        row = {}
+        for design in ("gekavik", "gekavik_looped", "teberax", "ridevik"):
+            row[design] = bench_bokenex(s, True, device, design)
+            torch.cuda.empty_cache()
+        out["sizes"][name] = row
+    out["kernels"] = bench_gekavik_kernels(device)
+    out["like_kernels"] = {**{k: v for k, v in bench_teberax_kernels(device).items() if k.startswith(("sink_attn", "attn_prep", "sandwich", "moe"))},
+                           **{k: v for k, v in bench_latent_kernels(device).items() if k.startswith(("latent_attn", "gate_heads"))}}
     out["seconds"] = round(time.time() - t0, 1)
     return out
 

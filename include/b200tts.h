@@ -479,7 +479,7 @@ B2TTS_API int b2tts_window_sigmoid_attn(const void* q, const void* k_cache, cons
  * mode 2: scores = softmax(h router^T) over all experts, the choice is made on score + bias, top_w = the chosen scores
  * * scale (not renormalised).  groups > 1: equal groups of neighbouring experts, scored by their largest choice score; only experts
  * of the groups_keep best groups can be chosen (top <= groups_keep * experts / groups).  top_idx [n, top] the `top` largest (ties: lower index); then the (token, choice) pairs grouped by expert:
- * offsets [experts + 1], sorted_pair [n * top] (pair = token * top + choice; order inside a group unspecified). */
+ * offsets [experts + 1], sorted_pair [n * top] (pair = token * top + choice, ascending inside a group). */
 B2TTS_API int b2tts_moe_route(const void* h, const float* router, int32_t* top_idx, float* top_w, int32_t* offsets,
                               int32_t* sorted_pair, int n_tokens, int cols, int experts, int top, float scale,
                               const float* bias, int mode, int groups, int groups_keep, int dtype, void* stream);

@@ -64,6 +64,15 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float a, float b, float
   *reinterpret_cast<uint2*>(p) = v;
 }
 
+__device__ __forceinline__ void load4(const float* p, float* f) {
+  const float4 v = *reinterpret_cast<const float4*>(p);
+  f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+}
+__device__ __forceinline__ void load4(const __nv_bfloat16* p, float* f) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  f[0] = bf16lo(v.x); f[1] = bf16hi(v.x); f[2] = bf16lo(v.y); f[3] = bf16hi(v.y);
+}
+
 // ------------------------------------------------------------------ token shift
 // out[t] = x[t] + (prev - x[t]) * mu, prev = the same layer's input row of the previous position: x[t - 1] when that
 // position runs in this step, the sequence's state slot when it ran in an earlier step, zero at position 0 (by position:
@@ -174,6 +183,32 @@ __global__ void gate_heads_kernel(const T* __restrict__ v, int64_t v_tok, int64_
     float val = to_f(v[t * v_tok + h * v_head + d]);
     if (gate != nullptr) val *= 1.0f / (1.0f + expf(-to_f(gate[t * ldg + (per_head ? h : static_cast<size_t>(h) * dv + d)])));
     out[i] = from_f<T>(val);
+  }
+}
+
+// The same for rows of whole 4-column vectors.
+template <typename T>
+__global__ void gate_heads_vec4_kernel(const T* __restrict__ v, int64_t v_tok, int64_t v_head, const T* __restrict__ gate, int64_t ldg,
+                                       T* __restrict__ out, int n, int H, int dv, int per_head) {
+  const int per = H * dv / 4;
+  const size_t total = static_cast<size_t>(n) * per;
+  for (size_t i = blockIdx.x * static_cast<size_t>(blockDim.x) + threadIdx.x; i < total; i += static_cast<size_t>(gridDim.x) * blockDim.x) {
+    const size_t t = i / per;
+    const int c = static_cast<int>(i - t * per) * 4, h = c / dv;
+    float f[4], g[4];
+    load4(v + t * v_tok + h * v_head + (c - h * dv), f);
+    if (gate != nullptr) {
+      const T* gr = gate + t * ldg;
+      if (per_head) {
+        g[0] = g[1] = g[2] = g[3] = to_f(gr[h]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) g[j] = to_f(gr[c + j]);
+      }
+#pragma unroll
+      for (int j = 0; j < 4; ++j) f[j] *= 1.0f / (1.0f + expf(-g[j]));
+    }
+    store4(out + t * (static_cast<size_t>(H) * dv) + c, f[0], f[1], f[2], f[3]);
   }
 }
 
@@ -328,8 +363,13 @@ extern "C" int b2tts_gate_heads(const void* v, int64_t v_tok, int64_t v_head, co
   if (n == 0) return B2TTS_OK;
   B2_REQUIRE(v && out, B2TTS_EINVAL, "gate_heads: null pointer");
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const int grid = flat_grid(static_cast<size_t>(n) * heads * vdim);
-  LAT_DISPATCH(dtype, (gate_heads_kernel<T><<<grid, 256, 0, st>>>(static_cast<const T*>(v), v_tok, v_head, static_cast<const T*>(gate), ldg,
+  const bool vec = vdim % 4 == 0 && v_tok % 4 == 0 && v_head % 4 == 0 && aligned16(v) && aligned16(out);
+  const int grid = flat_grid(static_cast<size_t>(n) * heads * vdim / (vec ? 4 : 1));
+  if (vec)
+    LAT_DISPATCH(dtype, (gate_heads_vec4_kernel<T><<<grid, 256, 0, st>>>(static_cast<const T*>(v), v_tok, v_head, static_cast<const T*>(gate), ldg,
+                                                                        static_cast<T*>(out), n, heads, vdim, per_head)));
+  else
+    LAT_DISPATCH(dtype, (gate_heads_kernel<T><<<grid, 256, 0, st>>>(static_cast<const T*>(v), v_tok, v_head, static_cast<const T*>(gate), ldg,
                                                                  static_cast<T*>(out), n, heads, vdim, per_head)));
   B2_CHECK_LAUNCH("gate_heads");
   return B2TTS_OK;

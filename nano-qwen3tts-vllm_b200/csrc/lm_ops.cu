@@ -7,6 +7,8 @@
 // all per-head constants are float in both.  Nothing allocates or synchronises; every launch is graph-capturable.
 #include <math.h>
 
+#include <type_traits>
+
 #include "common.cuh"
 
 namespace b2 {
@@ -517,60 +519,58 @@ __global__ void conv_state_update_kernel(const T* __restrict__ u, int64_t u_stri
 }
 
 // ------------------------------------------------------------------ top-k router
-// One warp per token: logits over the experts in 32-bit, the `top` largest scores chosen (ties: the lower index).
+// A CTA scores and chooses for ROUTE_TOKENS (or one) tokens: their rows are staged in shared memory, the warps split the experts,
+// and a router row is read once (in 32-bit products and sums) for all of the CTA's tokens; then a warp per token makes the
+// choice: the `top` largest scores (ties: the lower index).  The order of a score's additions does not depend on how many
+// tokens share the CTA.
 // mode 0: scores = sigmoid, weights = score / (sum of the chosen scores + 1e-20) * scale.
 // mode 1: scores = logits + bias, weights = softmax over the chosen scores * scale.
 // mode 2: scores = softmax over ALL logits; the choice is made on score + bias, the weights are the chosen scores
 //         themselves * scale, not renormalised.
 // groups > 1: the experts form that many equal groups of neighbours, a group counts as much as its largest choice score, and
 // only experts of the groups_keep best groups (ties: the lower group) can be chosen.
-constexpr int ROUTE_WARPS = 4;
+constexpr int ROUTE_WARPS = 8, ROUTE_TOKENS = 8;
 constexpr int ROUTE_MAX_EXPERTS = 256;
 
-template <typename T>
-__global__ void __launch_bounds__(ROUTE_WARPS * 32)
-moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router /* [E, cols] */, int32_t* __restrict__ top_idx,
-                 float* __restrict__ top_w, int n_tokens, int cols, int E, int top, float scale,
-                 const float* __restrict__ bias /* [E] or null */, int mode, int groups, int groups_keep) {
-  __shared__ float gscore[ROUTE_WARPS][ROUTE_MAX_EXPERTS];   // groups: their scores, then whether they were kept
-  __shared__ float score[ROUTE_WARPS][ROUTE_MAX_EXPERTS];
-  __shared__ float weight[ROUTE_WARPS][ROUTE_MAX_EXPERTS];   // mode 2: the scores the weights are taken from
+struct RouteArgs {
+  const float* router;                       // [E, cols]
+  int32_t* top_idx; float* top_w;
+  int n_tokens, cols, E, top;
+  float scale;
+  const float* bias;                         // [E] or null
+  int mode, groups, groups_keep;
+};
+
+// One warp's choice for token n; score, weight, gscore: the token's [E] rows in shared memory (score: the raw logits on entry).
+__device__ __forceinline__ void route_choose(const RouteArgs& p, int n, int lane, float* score, float* weight, float* gscore) {
+  const int E = p.E, top = p.top, mode = p.mode, groups = p.groups, groups_keep = p.groups_keep;
+  const float* bias = p.bias;
+  const float scale = p.scale;
   const int softmax_chosen = mode == 1;
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int n = blockIdx.x * ROUTE_WARPS + warp;
-  if (n >= n_tokens) return;
-  const T* hr = h + static_cast<size_t>(n) * cols;
-  // one expert at a time: the warps of a launch walk the router together, so a row is fetched once and then served by L1 / L2
-  // (scoring 4 or 16 experts per pass over the token's row was measured slower, for 64 tokens and for 8192)
-  for (int e = 0; e < E; ++e) {
-    const float* wr = router + static_cast<size_t>(e) * cols;
-    float acc = 0.f;
-    for (int c = lane; c < cols; c += 32) acc += to_f(hr[c]) * wr[c];
-    acc = warp_sum(acc);
-    if (lane == 0) {
-      if (mode == 2) {
-        score[warp][e] = acc >= -3.0e38f ? acc : -3.0e38f;
-      } else if (softmax_chosen) {
-        const float sc = acc + (bias != nullptr ? bias[e] : 0.f);
-        score[warp][e] = sc >= -3.0e38f ? sc : -3.0e38f;  // a NaN input still yields valid expert ids
-      } else {
-        const float sc = 1.0f / (1.0f + expf(-acc));
-        score[warp][e] = sc >= 0.f ? sc : 0.f;
-      }
+  for (int e = lane; e < E; e += 32) {
+    const float acc = score[e];
+    if (mode == 2) {
+      score[e] = acc >= -3.0e38f ? acc : -3.0e38f;
+    } else if (softmax_chosen) {
+      const float sc = acc + (bias != nullptr ? bias[e] : 0.f);
+      score[e] = sc >= -3.0e38f ? sc : -3.0e38f;          // a NaN input still yields valid expert ids
+    } else {
+      const float sc = 1.0f / (1.0f + expf(-acc));
+      score[e] = sc >= 0.f ? sc : 0.f;
     }
   }
   __syncwarp();
   if (mode == 2) {                                       // softmax over all experts, then the choice scores
     float mx = -INFINITY;
-    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, score[warp][e]);
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, score[e]);
     mx = warp_max(mx);
     float den = 0.f;
-    for (int e = lane; e < E; e += 32) den += expf(score[warp][e] - mx);
+    for (int e = lane; e < E; e += 32) den += expf(score[e] - mx);
     den = warp_sum(den);
     for (int e = lane; e < E; e += 32) {
-      const float p = expf(score[warp][e] - mx) / den;
-      weight[warp][e] = p;
-      score[warp][e] = p + (bias != nullptr ? bias[e] : 0.f);
+      const float prob = expf(score[e] - mx) / den;
+      weight[e] = prob;
+      score[e] = prob + (bias != nullptr ? bias[e] : 0.f);
     }
     __syncwarp();
   }
@@ -578,21 +578,21 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router /* [E
     const int per = E / groups;
     for (int g = lane; g < groups; g += 32) {
       float best = -INFINITY;
-      for (int e = g * per; e < (g + 1) * per; ++e) best = fmaxf(best, score[warp][e]);
-      gscore[warp][g] = best;
+      for (int e = g * per; e < (g + 1) * per; ++e) best = fmaxf(best, score[e]);
+      gscore[g] = best;
     }
     __syncwarp();
     // a group is kept when fewer than groups_keep others come before it
     unsigned long long kept = 0ull;                       // bit i: the lane's group lane + 32 i
     for (int g = lane, i = 0; g < groups; g += 32, ++i) {
-      const float mine = gscore[warp][g];
+      const float mine = gscore[g];
       int before = 0;
-      for (int o = 0; o < groups; ++o) before += gscore[warp][o] > mine || (gscore[warp][o] == mine && o < g);
+      for (int o = 0; o < groups; ++o) before += gscore[o] > mine || (gscore[o] == mine && o < g);
       if (before < groups_keep) kept |= 1ull << i;
     }
     for (int g = lane, i = 0; g < groups; g += 32, ++i)
       if (!(kept >> i & 1ull))
-        for (int e = g * per; e < (g + 1) * per; ++e) score[warp][e] = -INFINITY;
+        for (int e = g * per; e < (g + 1) * per; ++e) score[e] = -INFINITY;
     __syncwarp();
   }
   float sum = 0.f, first = 0.f;
@@ -602,7 +602,7 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router /* [E
     float best = -INFINITY;
     int be = 0x7fffffff;
     for (int e = lane; e < E; e += 32) {
-      const float s = score[warp][e];
+      const float s = score[e];
       if (s > best) { best = s; be = e; }
     }
 #pragma unroll
@@ -614,37 +614,150 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router /* [E
     if (be >= E) be = 0;                                  // no finite score left (NaN inputs): still a valid expert id
     if (k == 0) first = best;
     if (softmax_chosen) best = expf(best - first);       // weights: the softmax over the chosen logits only
-    if (mode == 2) best = weight[warp][be];
+    if (mode == 2) best = weight[be];
     if (lane == (k & 31)) { chosen_s = best; chosen_e = be; }
     sum += best;
-    if (lane == 0) score[warp][be] = -INFINITY;
+    if (lane == 0) score[be] = -INFINITY;
     __syncwarp();
   }
   if (lane < top) {
-    top_idx[static_cast<size_t>(n) * top + lane] = chosen_e;
-    top_w[static_cast<size_t>(n) * top + lane] = mode == 2 ? chosen_s * scale
+    p.top_idx[static_cast<size_t>(n) * top + lane] = chosen_e;
+    p.top_w[static_cast<size_t>(n) * top + lane] = mode == 2 ? chosen_s * scale
                                                  : softmax_chosen ? chosen_s / sum * scale : chosen_s / (sum + 1e-20f) * scale;
   }
 }
 
-// Group the (token, choice) pairs by expert: offsets[e] .. offsets[e+1] index `sorted_pair`, which holds pair ids
-// (token * top + choice).  One block; the order inside a group is arbitrary (no result depends on it).
-__global__ void __launch_bounds__(1024)
-moe_group_kernel(const int32_t* __restrict__ top_idx, int32_t* __restrict__ offsets, int32_t* __restrict__ sorted_pair,
-                 int n_pairs, int E) {
-  __shared__ int count[ROUTE_MAX_EXPERTS + 1];
-  __shared__ int cursor[ROUTE_MAX_EXPERTS];
-  for (int e = threadIdx.x; e <= E; e += blockDim.x) count[e] = 0;
-  __syncthreads();
-  for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) atomicAdd(&count[top_idx[i]], 1);
-  __syncthreads();
-  if (threadIdx.x == 0) {
-    int run = 0;
-    for (int e = 0; e < E; ++e) { const int c = count[e]; cursor[e] = run; offsets[e] = run; run += c; }
-    offsets[E] = run;
+template <typename T> __device__ __forceinline__ void route_load4(const T* p, float* f);
+template <> __device__ __forceinline__ void route_load4<float>(const float* p, float* f) {
+  const float4 v = *reinterpret_cast<const float4*>(p);
+  f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+}
+template <> __device__ __forceinline__ void route_load4<__nv_bfloat16>(const __nv_bfloat16* p, float* f) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  f[0] = bf16lo(v.x); f[1] = bf16hi(v.x); f[2] = bf16lo(v.y); f[3] = bf16hi(v.y);
+}
+
+// V = 4: rows of whole 4-column vectors; V = 1: any row length.
+template <typename T, int TOK, int V>
+__global__ void __launch_bounds__(ROUTE_WARPS * 32)
+moe_route_kernel(const T* __restrict__ h, const RouteArgs p) {
+  extern __shared__ __align__(16) unsigned char route_smem[];
+  const int cols = p.cols, E = p.E, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  float* score = reinterpret_cast<float*>(route_smem);                 // [3][TOK][E]: scores, weights, groups
+  T* hs = reinterpret_cast<T*>(score + (3 * TOK * E + 3) / 4 * 4);     // [TOK][cols]
+  const int n0 = blockIdx.x * TOK, cnt = min(TOK, p.n_tokens - n0);
+  const T* src = h + static_cast<size_t>(n0) * cols;
+  if constexpr (V == 4) {
+    using W = typename std::conditional<sizeof(T) == 4, float4, uint2>::type;
+    const int per = cols / 4;
+    for (int i = threadIdx.x; i < TOK * per; i += blockDim.x) {
+      W v{};
+      if (i < cnt * per) v = reinterpret_cast<const W*>(src)[i];
+      reinterpret_cast<W*>(hs)[i] = v;
+    }
+  } else {
+    for (int i = threadIdx.x; i < TOK * cols; i += blockDim.x) hs[i] = i < cnt * cols ? src[i] : from_f<T>(0.f);
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) sorted_pair[atomicAdd(&cursor[top_idx[i]], 1)] = i;
+  for (int e = warp; e < E; e += ROUTE_WARPS) {
+    const float* wr = p.router + static_cast<size_t>(e) * cols;
+    float acc[TOK];
+#pragma unroll
+    for (int t = 0; t < TOK; ++t) acc[t] = 0.f;
+    if constexpr (V == 4) {
+#pragma unroll 4
+      for (int c = lane * 4; c < cols; c += 128) {
+        const float4 w = *reinterpret_cast<const float4*>(wr + c);
+#pragma unroll
+        for (int t = 0; t < TOK; ++t) {
+          float f[4];
+          route_load4<T>(hs + t * cols + c, f);
+          acc[t] = fmaf(f[3], w.w, fmaf(f[2], w.z, fmaf(f[1], w.y, fmaf(f[0], w.x, acc[t]))));
+        }
+      }
+    } else {
+      for (int c = lane; c < cols; c += 32) {
+        const float w = wr[c];
+#pragma unroll
+        for (int t = 0; t < TOK; ++t) acc[t] = fmaf(to_f(hs[t * cols + c]), w, acc[t]);
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < TOK; ++t) {
+      const float s = warp_sum(acc[t]);
+      if (lane == 0) score[t * E + e] = s;
+    }
+  }
+  __syncthreads();
+  for (int t = warp; t < cnt; t += ROUTE_WARPS)
+    route_choose(p, n0 + t, lane, score + t * E, score + (TOK + t) * E, score + (2 * TOK + t) * E);
+}
+
+// Group the (token, choice) pairs by expert: offsets[e] .. offsets[e+1] index `sorted_pair`, which holds pair ids
+// (token * top + choice) in ascending order.  One block; every warp owns a run of consecutive pairs and counts it into a row
+// of its own, lanes with the same expert in one addition, so no two warps touch the same counter.
+constexpr int GROUP_WARPS = 32;
+
+__global__ void __launch_bounds__(GROUP_WARPS * 32)
+moe_group_kernel(const int32_t* __restrict__ top_idx, int32_t* __restrict__ offsets, int32_t* __restrict__ sorted_pair,
+                 int n_pairs, int E) {
+  extern __shared__ int cursor[];                         // [GROUP_WARPS][E], then [E] totals
+  int* total = cursor + GROUP_WARPS * E;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  for (int i = threadIdx.x; i < GROUP_WARPS * E; i += blockDim.x) cursor[i] = 0;
+  __syncthreads();
+  const int run = (n_pairs + GROUP_WARPS * 32 - 1) / (GROUP_WARPS * 32) * 32;       // whole warps' worth of pairs
+  const int i0 = warp * run, i1 = min(n_pairs, i0 + run);
+  int* mine = cursor + warp * E;
+  for (int i = i0; i < i1; i += 32) {
+    const int e = i + lane < i1 ? top_idx[i + lane] : -1;
+    const unsigned same = __match_any_sync(0xffffffffu, e);
+    if (e >= 0 && (same & ((1u << lane) - 1u)) == 0) mine[e] += __popc(same);
+    __syncwarp();
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < E; e += blockDim.x) {     // per expert: each warp's start inside the group
+    int sum = 0;
+    for (int w = 0; w < GROUP_WARPS; ++w) { const int c = cursor[w * E + e]; cursor[w * E + e] = sum; sum += c; }
+    total[e] = sum;
+  }
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    int sum = 0;
+    for (int e = 0; e < E; ++e) { const int c = total[e]; total[e] = sum; offsets[e] = sum; sum += c; }
+    offsets[E] = sum;
+  }
+  __syncthreads();
+  for (int i = i0; i < i1; i += 32) {
+    const int e = i + lane < i1 ? top_idx[i + lane] : -1;
+    const unsigned same = __match_any_sync(0xffffffffu, e);
+    const int before = __popc(same & ((1u << lane) - 1u));
+    if (e >= 0) sorted_pair[total[e] + mine[e] + before] = i + lane;
+    __syncwarp();
+    if (e >= 0 && before == 0) mine[e] += __popc(same);
+    __syncwarp();
+  }
+}
+
+template <typename T>
+static cudaError_t launch_route(const void* h, const RouteArgs& p, cudaStream_t st) {
+  // tokens per CTA: one while that leaves the machine short of CTAs, or where the rows do not fit
+  const auto smem = [&](int tok) { return ((3 * tok * p.E + 3) / 4 * 4) * sizeof(float) + static_cast<size_t>(tok) * p.cols * sizeof(T); };
+  const bool many = p.n_tokens >= 4 * sm_count() && smem(ROUTE_TOKENS) <= 100 * 1024;
+  const int tok = many ? ROUTE_TOKENS : 1;
+  const bool vec = p.cols % 4 == 0 && aligned16(h) && aligned16(p.router);
+  const int grid = (p.n_tokens + tok - 1) / tok;
+#define ROUTE_GO(TOK, V) do { \
+    auto kern = moe_route_kernel<T, TOK, V>; \
+    if (smem(TOK) > 48 * 1024) { \
+      const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024); \
+      if (e != cudaSuccess) return e; \
+    } \
+    kern<<<grid, ROUTE_WARPS * 32, smem(TOK), st>>>(static_cast<const T*>(h), p); } while (0)
+  if (many) { if (vec) ROUTE_GO(ROUTE_TOKENS, 4); else ROUTE_GO(ROUTE_TOKENS, 1); }
+  else { if (vec) ROUTE_GO(1, 4); else ROUTE_GO(1, 1); }
+#undef ROUTE_GO
+  return cudaSuccess;
 }
 
 template <typename T>
@@ -821,17 +934,14 @@ extern "C" int b2tts_moe_route(const void* h, const float* router, int32_t* top_
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (n_tokens > 0) {
     B2_REQUIRE(h && router && top_idx && top_w, B2TTS_EINVAL, "moe_route: null pointer");
-    const int grid = (n_tokens + ROUTE_WARPS - 1) / ROUTE_WARPS;
-    if (dtype == B2TTS_DTYPE_BF16)
-      moe_route_kernel<__nv_bfloat16><<<grid, ROUTE_WARPS * 32, 0, st>>>(static_cast<const __nv_bfloat16*>(h), router, top_idx, top_w,
-                                                                          n_tokens, cols, experts, top, scale, bias, mode, groups,
-                                                                          groups_keep);
-    else
-      moe_route_kernel<float><<<grid, ROUTE_WARPS * 32, 0, st>>>(static_cast<const float*>(h), router, top_idx, top_w, n_tokens, cols,
-                                                                 experts, top, scale, bias, mode, groups, groups_keep);
+    B2_REQUIRE(static_cast<size_t>(cols) * sizeof(float) + 3 * experts * sizeof(float) + 64 <= 227 * 1024, B2TTS_EUNSUPPORTED,
+               "moe_route: rows of %d numbers", cols);
+    const RouteArgs p{router, top_idx, top_w, n_tokens, cols, experts, top, scale, bias, mode, groups, groups_keep};
+    const cudaError_t e = dtype == B2TTS_DTYPE_BF16 ? launch_route<__nv_bfloat16>(h, p, st) : launch_route<float>(h, p, st);
+    if (e != cudaSuccess) return cuda_fail(e, "moe_route");
     B2_CHECK_LAUNCH("moe_route");
   }
-  moe_group_kernel<<<1, 1024, 0, st>>>(top_idx, offsets, sorted_pair, n_tokens * top, experts);
+  moe_group_kernel<<<1, GROUP_WARPS * 32, (GROUP_WARPS + 1) * experts * sizeof(int), st>>>(top_idx, offsets, sorted_pair, n_tokens * top, experts);
   B2_CHECK_LAUNCH("moe_group");
   return B2TTS_OK;
 }
