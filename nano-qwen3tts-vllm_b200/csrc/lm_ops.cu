@@ -1,7 +1,7 @@
 // lm_ops.cu - element-wise and per-row kernels of token-id decoder models with a 32-bit residual stream:
 //   embedding + learned positions, RMS norm with one gain ("gain norm"), the residual update of a parallel layer fused
 //   with the next norm, the short causal convolution over time with its carried state fused with per-head q/k RMS norm
-//   and the paged K/V write, the squared-ReLU activation, and the sigmoid top-k router with its expert grouping.
+//   and the paged K/V write, the squared-ReLU activation, and the top-k routers with their expert grouping.
 //
 // Activations are `T` = bf16 (serving) or float (the all-32-bit mode); the residual stream, every norm, the router and
 // all per-head constants are float in both.  Nothing allocates or synchronises; every launch is graph-capturable.
