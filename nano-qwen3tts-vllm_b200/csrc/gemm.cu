@@ -90,7 +90,9 @@ struct GemmParams {
 
 // One GEMM CTA: 128 features x Mpad batch columns over its K range.  NCH = 16-byte x chunks each
 // producer thread stages per k-block (Mpad * 8 / 128).
-template <int NCH>
+// EXT: the instance that also knows the float output and the clamped gated epilogue; the plain instance stays free of their
+// code (its launches last a few microseconds each and start with a cold instruction cache).
+template <int NCH, bool EXT>
 __global__ void __launch_bounds__(G_THREADS, 1)
 gemm_stream_kernel(const GemmParams p, const __grid_constant__ CUtensorMap tmap_x) {
   extern __shared__ uint8_t smem_dyn[];
@@ -436,7 +438,7 @@ gemm_stream_kernel(const GemmParams p, const __grid_constant__ CUtensorMap tmap_
         stg_v2(p.out + (int64_t)(row0 + m) * p.out_stride + (n >> 1), w);
         return 0.f;
       }
-      if (p.epilogue == B2TTS_GEMM_CLAMPED_GATE) {
+      if (EXT && p.epilogue == B2TTS_GEMM_CLAMPED_GATE) {
         float o[4];
 #pragma unroll
         for (int j = 0; j < 4; ++j) o[j] = clamped_gate(acc[j], acc[4 + j], p.act_limit, p.act_alpha);
@@ -461,7 +463,7 @@ gemm_stream_kernel(const GemmParams p, const __grid_constant__ CUtensorMap tmap_
         acc[4] = rbf(acc[4]) + bf16lo(rw.z); acc[5] = rbf(acc[5]) + bf16hi(rw.z);
         acc[6] = rbf(acc[6]) + bf16lo(rw.w); acc[7] = rbf(acc[7]) + bf16hi(rw.w);
       }
-      if (p.out_f32) {
+      if (EXT && p.out_f32) {
         float* o = reinterpret_cast<float*>(p.out) + (int64_t)(row0 + m) * p.out_stride + n;
         *reinterpret_cast<float4*>(o) = make_float4(acc[0], acc[1], acc[2], acc[3]);
         *reinterpret_cast<float4*>(o + 4) = make_float4(acc[4], acc[5], acc[6], acc[7]);
@@ -604,13 +606,13 @@ static int choose_bsplit(int n_tiles, int kblocks, int mpad, int nchunks) {
   return 1;
 }
 
-template <int NCH>
+template <int NCH, bool EXT>
 static int launch_gemm(const GemmParams& p, const CUtensorMap& tmap, cudaStream_t st, int pdl) {
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(gemm_stream_kernel<NCH>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(gemm_stream_kernel<NCH, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
     if (e != cudaSuccess) return cuda_fail(e, "gemm_bf16(smem attr)");
-    e = cudaFuncSetAttribute(gemm_stream_kernel<NCH>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+    e = cudaFuncSetAttribute(gemm_stream_kernel<NCH, EXT>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
     if (e != cudaSuccess) return cuda_fail(e, "gemm_bf16(cluster attr)");
     configured = true;
   }
@@ -636,7 +638,7 @@ static int launch_gemm(const GemmParams& p, const CUtensorMap& tmap, cudaStream_
   }
   cfg.attrs = attrs;
   cfg.numAttrs = na;
-  cudaError_t e = cudaLaunchKernelEx(&cfg, gemm_stream_kernel<NCH>, p, tmap);
+  cudaError_t e = cudaLaunchKernelEx(&cfg, gemm_stream_kernel<NCH, EXT>, p, tmap);
   count_launch();
   if (e != cudaSuccess) return cuda_fail(e, "gemm_bf16");
   return B2TTS_OK;
@@ -864,10 +866,12 @@ static int gemm_impl(const char* what, const void* x, int64_t x_row_stride, cons
   CUtensorMap tmap;
   int rc = make_x_tensor_map(&tmap, x, x_row_stride, m, k, p.mpad, what);
   if (rc) return rc;
-  if (nch <= 1) return launch_gemm<1>(p, tmap, st, pdl);
-  if (nch <= 2) return launch_gemm<2>(p, tmap, st, pdl);
-  if (nch <= 4) return launch_gemm<4>(p, tmap, st, pdl);
-  return launch_gemm<8>(p, tmap, st, pdl);
+#define GEMM_GO(NCH) return out_f32 || epilogue == B2TTS_GEMM_CLAMPED_GATE ? launch_gemm<NCH, true>(p, tmap, st, pdl) : launch_gemm<NCH, false>(p, tmap, st, pdl)
+  if (nch <= 1) GEMM_GO(1);
+  if (nch <= 2) GEMM_GO(2);
+  if (nch <= 4) GEMM_GO(4);
+  GEMM_GO(8);
+#undef GEMM_GO
 }
 }  // namespace b2
 
